@@ -106,6 +106,18 @@ class LayerNormSpec:
 
 
 @dataclass(frozen=True)
+class GroupedRMSNormSpec:
+    """Root-mean-square norm in groups: the row is cut into ``groups`` equal parts of neighbours, each part is divided
+    by its own ``sqrt(mean(part^2) + eps)``, then the whole row is multiplied by a weight ``[size]``."""
+
+    size: int
+    eps: float
+    groups: int = 1
+    weight: str = "weight"
+    kind: str = "grouped_rmsnorm"
+
+
+@dataclass(frozen=True)
 class AttentionNames:
     """Checkpoint names of an attention layer's tensors, behind the layer's prefix.  An architecture's
     configuration sets them; the part has none of its own."""
@@ -186,8 +198,8 @@ class LatentAttentionSpec:
     gives ``kv_rank + rot_dim`` numbers per token: the first ``kv_rank``, divided by their root mean square (``eps``
     inside the root) and multiplied by a weight, are the latent ``c``; the last ``rot_dim``, rotated, are a key part
     all heads share.  Head h's unrotated key is ``Uk_h c`` and its value ``Uv_h c`` (``value_dim`` numbers); the score
-    is ``(q_plain . k_plain + q_rot . k_rot) * softmax_scale``.  ``position`` (variant ``"interleaved"``) turns the
-    first ``position.dim`` of the rotated dims.  ``sink``: one learned score per head joins the softmax's
+    is ``(q_plain . k_plain + q_rot . k_rot) * softmax_scale``.  ``position`` (variant ``"interleaved"`` or
+    ``"half_partial"``) turns the first ``position.dim`` of the rotated dims.  ``sink``: one learned score per head joins the softmax's
     denominator with no key and no value.  Only ``c`` and the rotated key part are kept per token."""
 
     hidden: int
@@ -248,7 +260,11 @@ class RoutedExpertsSpec:
     score: its largest choice score); the WEIGHTS are the chosen experts' ``s`` over their sum (+ 1e-20), times
     ``scale``.  ``shared``: a gated feed-forward of the same form that every token runs, added to the sum.  Expert e's
     tensors are ``prefix + expert.format(e) + gate / up / down``; identity experts are the router's last outputs and
-    have no tensors."""
+    have no tensors.
+
+    ``scores`` ``"sigmoid"``: ``s = sigmoid(z)`` element by element instead of the softmax.  ``correction`` None: experts are
+    chosen by ``s`` itself.  ``renormalize`` False: the weights are the chosen ``s`` times ``scale`` as they are.
+    ``weight_on`` ``"input"``: a weight multiplies its expert's input instead of its output, ``expert(w x)``."""
 
     hidden: int
     intermediate: int
@@ -261,7 +277,10 @@ class RoutedExpertsSpec:
     activation: str = "silu"
     shared: Optional["GatedMLPSpec"] = None
     router: str = "router"
-    correction: str = "correction"
+    correction: Optional[str] = "correction"
+    scores: str = "softmax"
+    renormalize: bool = True
+    weight_on: str = "output"
     expert: str = "e{}."
     names: GatedMLPNames = GatedMLPNames(gate="gate", up="up", down="down")
     kind: str = "routed_experts"
@@ -353,13 +372,14 @@ class HeadAttentionNames:
     gate: str = "g"
     bias: str = ".b"
     sink: str = "sink"
+    score_bias: str = "pb"
 
 
 @dataclass(frozen=True)
 class HeadAttentionSpec:
     """Causal grouped-query attention (a *mixer*) whose q and k heads are normed (RMS over the head, one weight
     for all heads, ``eps``) before an optional rotation of the first ``position.dim`` dims of each head (variant
-    ``"half_partial"``).  Each of the following is an option: biases on the input projections (``bias_in``) and on
+    ``"half_partial"`` or ``"interleaved"``).  Each of the following is an option: biases on the input projections (``bias_in``) and on
     the output projection (``bias_out``); ``values_from_keys``: there is no value projection, a token's value is its
     key as projected (with bias, before norm and rotation); ``window`` of W: a query at p sees keys p - W + 1 .. p;
     ``unit_sink``: the softmax's denominator has one more term of score 0 and no value; ``sink``: that term's score is a
@@ -367,7 +387,12 @@ class HeadAttentionSpec:
     (with a window): a query also sees the sequence's first F keys, however far back; ``softcap`` c: a score becomes
     ``c tanh(score / c)`` after the scale; ``slope_exponent`` c: head h of H takes ``2^(-c (h + 1) / H)`` times the
     distance to a key off its score; ``head_gate``: a head's output times ``sigmoid`` of one number per head projected
-    from the mixer's input."""
+    from the mixer's input; ``channel_gate``: the same with one number per channel (tensor ``names.gate`` [n_heads *
+    value_dim, hidden]); ``qk_norm_over`` ``"projection"``: q and k are normed over all their heads' rows at once, with
+    weights of that size, before they are split into heads; ``value_norm``: every value head is divided by its root mean
+    square (``eps``, no weight) and cached so; ``chunk`` of C: a query at p sees only keys of its own chunk, p - p mod C
+    .. p, chunks counted from the sequence's start; ``weights`` ``"sigmoid"``: no softmax, the weight of a visible key is
+    ``sigmoid(score + z_h)`` with a learned number per head (tensor ``names.score_bias`` [n_heads])."""
 
     hidden: int
     n_heads: int
@@ -388,6 +413,11 @@ class HeadAttentionSpec:
     sink: bool = False
     keep_first: int = 0
     softcap: Optional[float] = None
+    channel_gate: bool = False
+    qk_norm_over: str = "head"
+    value_norm: bool = False
+    chunk: Optional[int] = None
+    weights: str = "softmax"
     names: HeadAttentionNames = HeadAttentionNames()
     kind: str = "head_attention"
 
@@ -517,6 +547,21 @@ class PostNormLayerSpec:
     mixer_scale: Optional[str] = None
     feed_forward_scale: Optional[str] = None
     kind: str = "postnorm"
+
+
+@dataclass(frozen=True)
+class SumNormLayerSpec:
+    """A layer whose norms take the stream WITH the sublayer's output in it: ``h <- N1(alpha h + mixer(h))``, then, if it
+    has a feed-forward, ``h <- N2(alpha h + ff(h))``.  The sublayers read the stream itself.  The norms (RMS norms in
+    groups) have their tensors at ``prefix + <spec.weight>``."""
+
+    prefix: str
+    mixer: object
+    mixer_norm: GroupedRMSNormSpec
+    feed_forward: Optional[object] = None
+    feed_forward_norm: Optional[GroupedRMSNormSpec] = None
+    alpha: float = 1.0
+    kind: str = "sum_norm"
 
 
 @dataclass(frozen=True)

@@ -17,8 +17,12 @@
 // A scheduler warp takes the items and looks up what they need (lengths, page numbers) ahead of time; a
 // TMA warp requests an item's key blocks and then its value blocks, in that order, into one ring;
 // four warps do the arithmetic.
+// MODE: AF_PLAIN, a softmax over every earlier key; AF_CHUNK, over the keys of the query's chunk; AF_SIGMOID, sigmoid
+// weights over those (or all) keys.
 // The reference's single-token path: src/detllm/ops/fused_attn.py:47-115.
 #pragma once
+
+enum { AF_PLAIN = 0, AF_CHUNK = 1, AF_SIGMOID = 2 };
 
 #define AF_THREADS 192
 #define AF_MAX_RUN_BLOCKS 8
@@ -90,7 +94,7 @@ struct AttnFewLayout {
     __host__ __device__ int total() const { return need() + 1024; }
 };
 
-template <int HD>
+template <int HD, int MODE>
 __global__ void __launch_bounds__(AF_THREADS, 2)
 attention_few_rows_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                           AttnTcArgs a, const T* __restrict__ q, int slots, int n_tiles) {
@@ -145,7 +149,7 @@ attention_few_rows_kernel(const __grid_constant__ CUtensorMap map_k, const __gri
         prev.n_runs = 0; pending.n_runs = 0;
         int prev_st = 0, prev_parity = 0;
         for (int qn = 0; ok; ++qn) {
-            int item = -1, tile = 0, hg = 0, run = 0, seq = 0, tstart = 0, n_runs = 0, nb_tile = 0, toks_valid = 0, p_first = 0;
+            int item = -1, tile = 0, hg = 0, run = 0, seq = 0, tstart = 0, n_runs = 0, nb_tile = 0, toks_valid = 0, p_first = 0, run_lo = 0;
             for (;;) {
                 if (qn == 0 && !waited && item == -1) {
                     item = blockIdx.x;
@@ -163,7 +167,9 @@ attention_few_rows_kernel(const __grid_constant__ CUtensorMap map_k, const __gri
                 toks_valid = min(a.rows_cap >> gs, q_len - tstart);
                 p_first = a.q_start[seq] + tstart;
                 nb_tile = (p_first + toks_valid - 1) / AP_BN + 1;
-                n_runs = (nb_tile + R - 1) / R;
+                // (runs wholly before the chunk of the tile's first row are left out; a tile's runs are counted from the first that is not)
+                if (MODE != AF_PLAIN) run_lo = (attn_first_seen(a, p_first) / AP_BN) / R;
+                n_runs = (nb_tile + R - 1) / R - run_lo;
                 if (run < n_runs) break;
                 item = -2;                                       // (passed over: the next one comes from the counter)
             }
@@ -205,7 +211,7 @@ attention_few_rows_kernel(const __grid_constant__ CUtensorMap map_k, const __gri
             if (!ok) break;
             volatile AttnFewItem* d = items + st;
             if (item >= 0) {
-                const int b_first = run * R, nb = min(R, nb_tile - b_first);
+                const int b_first = (run + run_lo) * R, nb = min(R, nb_tile - b_first);
                 if (lane < nb) d->pages[lane] = a.table[(size_t)a.slots[seq] * a.table_stride + b_first + lane];
                 if (lane == 0) {
                     d->tile = tile; d->hg = hg; d->run = run; d->n_runs = n_runs;
@@ -384,6 +390,9 @@ attention_few_rows_kernel(const __grid_constant__ CUtensorMap map_k, const __gri
                 if (lane == 0) attn_stamp(11 + 3 * warp);
                 const int key0 = (b_first + bl) * AP_BN;
                 const int vis_lo = p_first + (r_lo >> gs) - key0, vis_hi = p_first + (r_hi >> gs) - key0;   // columns up to here count
+                // (columns below these lie before the row's chunk)
+                const int fst_lo = MODE == AF_CHUNK ? attn_first_seen(a, p_first + (r_lo >> gs)) - key0 : 0;
+                const int fst_hi = MODE == AF_CHUNK ? attn_first_seen(a, p_first + (r_hi >> gs)) - key0 : 0;
                 float mx_lo = -INFINITY, mx_hi = -INFINITY;
 #pragma unroll
                 for (int nt = 0; nt < 8; ++nt) {
@@ -396,12 +405,19 @@ attention_few_rows_kernel(const __grid_constant__ CUtensorMap map_k, const __gri
                         float* dst = s_sm + (r_hi * AF_MAX_RUN_BLOCKS + bl) * AF_S_STRIDE + col;
                         dst[0] = acc[nt][2]; dst[1] = acc[nt][3];
                     }
+                    if (MODE == AF_SIGMOID) continue;             // (no maximum is taken)
+                    if (MODE == AF_CHUNK) {
+                        if (col < fst_lo) acc[nt][0] = -INFINITY;
+                        if (col + 1 < fst_lo) acc[nt][1] = -INFINITY;
+                        if (col < fst_hi) acc[nt][2] = -INFINITY;
+                        if (col + 1 < fst_hi) acc[nt][3] = -INFINITY;
+                    }
                     mx_lo = fmaxf(mx_lo, fmaxf(col > vis_lo ? -INFINITY : acc[nt][0], col + 1 > vis_lo ? -INFINITY : acc[nt][1]));
                     mx_hi = fmaxf(mx_hi, fmaxf(col > vis_hi ? -INFINITY : acc[nt][2], col + 1 > vis_hi ? -INFINITY : acc[nt][3]));
                 }
                 mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 1)); mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 2));
                 mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 1)); mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 2));
-                if (tig == 0) {
+                if (MODE != AF_SIGMOID && tig == 0) {
                     if (r_lo < rows_valid) mblk_sm[r_lo * AF_MAX_RUN_BLOCKS + bl] = __fmul_rn(mx_lo, a.scale_log2);
                     if (r_hi < rows_valid) mblk_sm[r_hi * AF_MAX_RUN_BLOCKS + bl] = __fmul_rn(mx_hi, a.scale_log2);
                 }
@@ -419,18 +435,23 @@ attention_few_rows_kernel(const __grid_constant__ CUtensorMap map_k, const __gri
             const bool live = t_bl < nb;
             const float* s_row = s_sm + (t_row * AF_MAX_RUN_BLOCKS + (live ? t_bl : 0)) * AF_S_STRIDE;
             const int visible = p_first + (t_row >> gs) - (b_first + t_bl) * AP_BN;
+            const int first = MODE == AF_PLAIN ? 0 : attn_first_seen(a, p_first + (t_row >> gs)) - (b_first + t_bl) * AP_BN;
+            const float neg_scale = -a.scale_log2;
+            const float neg_bias = MODE == AF_SIGMOID ? -__fmul_rn(dry ? 0.f : a.score_bias[head0 + (t_row & (gp - 1))], 1.4426950408889634f) : 0.f;
             // where the running maximum stands when this block is reached, and whether this block moves it
-            float mb[AF_MAX_RUN_BLOCKS];
-#pragma unroll
-            for (int i = 0; i < AF_MAX_RUN_BLOCKS; ++i) mb[i] = i < nb ? mblk_sm[t_row * AF_MAX_RUN_BLOCKS + i] : -INFINITY;
-            float m_ref = -INFINITY, m_before = -INFINITY;
+            float m_ref = MODE == AF_SIGMOID ? 0.f : -INFINITY, m_before = -INFINITY;
             bool moved = false;
+            if (MODE != AF_SIGMOID) {
+                float mb[AF_MAX_RUN_BLOCKS];
 #pragma unroll
-            for (int i = 0; i < AF_MAX_RUN_BLOCKS; ++i) {
-                if (i <= t_bl) {
-                    moved = mb[i] > m_ref + AP_RESCALE_STEP;
-                    m_before = m_ref;
-                    if (moved) m_ref = mb[i];
+                for (int i = 0; i < AF_MAX_RUN_BLOCKS; ++i) mb[i] = i < nb ? mblk_sm[t_row * AF_MAX_RUN_BLOCKS + i] : -INFINITY;
+#pragma unroll
+                for (int i = 0; i < AF_MAX_RUN_BLOCKS; ++i) {
+                    if (i <= t_bl) {
+                        moved = mb[i] > m_ref + AP_RESCALE_STEP;
+                        m_before = m_ref;
+                        if (moved) m_ref = mb[i];
+                    }
                 }
             }
             const float alpha = moved ? exp2f(m_before - m_ref) : 1.f;
@@ -442,12 +463,13 @@ attention_few_rows_kernel(const __grid_constant__ CUtensorMap map_k, const __gri
             for (int i0 = 0; i0 < AP_BN / 4; i0 += 4) {
                 float sc[4];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) sc[i] = (live && 4 * (i0 + i) + u <= visible) ? s_row[4 * (i0 + i) + u] : -INFINITY;
+                for (int i = 0; i < 4; ++i)
+                    sc[i] = (live && 4 * (i0 + i) + u <= visible && (MODE == AF_PLAIN || 4 * (i0 + i) + u >= first)) ? s_row[4 * (i0 + i) + u] : -INFINITY;
                 __nv_bfloat16 pb[4];
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
-                    const float pj = ex2_hw(__fmaf_rn(sc[i], a.scale_log2, neg_m));
-                    sum = __fadd_rn(sum, pj);
+                    const float pj = MODE == AF_SIGMOID ? sigmoid_weight(sc[i], neg_scale, neg_bias) : ex2_hw(__fmaf_rn(sc[i], a.scale_log2, neg_m));
+                    if (MODE != AF_SIGMOID) sum = __fadd_rn(sum, pj);
                     pb[i] = __float2bfloat16_rn(pj);
                 }
                 if (live) {
@@ -598,7 +620,7 @@ attention_few_rows_kernel(const __grid_constant__ CUtensorMap map_k, const __gri
                 float M = -INFINITY, L = 0.f, a_, b_;
                 fold_coeffs(M, L, mfin_sm[r], lfin_sm[r], a_, b_);
                 const float sa = a.sink ? fold_sink(a.sink, head0 + (r & (gp - 1)), M, L) : 1.0f;
-                const float inv = __fdiv_rn(1.0f, L);
+                const float inv = MODE == AF_SIGMOID ? 1.0f : __fdiv_rn(1.0f, L);
                 T* orow = a.out + ((size_t)(tok0 + (r >> gs)) * a.n_q + head0 + (r & (gp - 1))) * HD;
 #pragma unroll
                 for (int nt = 0; nt < NT; ++nt) {
@@ -643,7 +665,7 @@ static bool attention_few_rows_can(int hd, int rows_cap, int run_blocks, int max
            groups <= AF_WORK_COUNTER;
 }
 
-template <int HD>
+template <int HD, int MODE>
 static int launch_attention_few_rows(const CUtensorMap& mk, const CUtensorMap& mv, const AttnTcArgs& a, const T* q,
                                      int n_tiles, cudaStream_t stream) {
     static int configured = 0, n_sm = 0;
@@ -659,12 +681,12 @@ static int launch_attention_few_rows(const CUtensorMap& mk, const CUtensorMap& m
     const int bytes = attention_few_rows_plan(HD, a.rows_cap, items, n_sm, &slots, &per_sm);
     IDM_REQUIRE(slots >= 4, "attention_few_rows: no room for the ring (%d rows)", a.rows_cap);
     if (configured < bytes) {
-        cudaError_t e = cudaFuncSetAttribute(attention_few_rows_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+        cudaError_t e = cudaFuncSetAttribute(attention_few_rows_kernel<HD, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
         IDM_REQUIRE(e == cudaSuccess, "attention_few_rows: cannot get %d bytes of shared memory: %s", bytes, cudaGetErrorString(e));
         configured = bytes;
     }
     const int grid = (int)(items < (long long)per_sm * n_sm ? items : (long long)per_sm * n_sm);
-    idm_launch(attention_few_rows_kernel<HD>, dim3(grid), dim3(AF_THREADS), (size_t)bytes, stream, mk, mv, a, q, slots, n_tiles);
+    idm_launch(attention_few_rows_kernel<HD, MODE>, dim3(grid), dim3(AF_THREADS), (size_t)bytes, stream, mk, mv, a, q, slots, n_tiles);
     IDM_LAUNCH_CHECK("attention_few_rows");
     return 0;
 }

@@ -5,7 +5,9 @@
 // A query at position p of sequence s sees keys j with max(0, p - window + 1) <= j <= p
 // (window <= 0: all j <= p), the slot-causal rule of src/detllm/model.py:259-266; with keep_first > 0 also the
 // keys j < keep_first, however far back they lie (the blocks of 32 that hold them are walked first, then the
-// window's).  softcap > 0 bounds a score: cap * tanh(score / cap), after the scale and before the softmax.
+// window's).  With chunk > 0 it sees the keys of its own chunk only, p - p % chunk <= j <= p (chunks counted from the
+// sequence's start).  softcap > 0 bounds a score: cap * tanh(score / cap), after the scale and before the softmax.
+// With score_bias there is no softmax: a visible key's weight is sigmoid(score + score_bias[head]) and nothing is divided.
 // Keys are walked in blocks of 32 aligned to absolute positions; inside a block lane i
 // scores key j0 + i; masked lanes contribute exactly 0 and are left out of the maximum
 // (the float analogue of the reference's integer sentinel, src/detllm/ops/di_softmax.py:45-58);
@@ -34,6 +36,8 @@ struct AttnArgs {
     int gate_per_head;            // the gate is one number per head: gate[t * gate_stride + head]
     float softcap;                // > 0: score <- softcap * tanh(score / softcap)
     int keep_first;               // > 0: keys j < keep_first are seen from any distance
+    int chunk;                    // > 0: only keys of the query's own chunk of so many positions are seen
+    const float* score_bias;      // [n_q] or null: the weights are sigmoid(score + score_bias[head]), not a softmax
 };
 
 #define AG_WARPS 4
@@ -53,7 +57,7 @@ __global__ void __launch_bounds__(AG_WARPS * 32) attention_generic_kernel(AttnAr
     __syncwarp();
     const int pos = a.positions[t], s = a.token_seq[t], slot = a.slots[s];
     const int first_new = a.k_new ? a.q_start[s] : 0x7fffffff, tok0 = a.cu_q[s];
-    const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+    const int lo = a.chunk > 0 ? pos - pos % a.chunk : a.window > 0 ? max(0, pos - a.window + 1) : 0;
     // a sink is a key of score sink[head] (not scaled) whose value is zero: the sums start from it
     float m = a.sink ? a.sink[head] : -INFINITY, l = a.sink ? 1.f : 0.f;
     float acc[IDM_MAX_HEAD_DIM / 32];
@@ -90,13 +94,18 @@ __global__ void __launch_bounds__(AG_WARPS * 32) attention_generic_kernel(AttnAr
             if (a.softcap > 0.f) sc = a.softcap * tanhf(sc / a.softcap);
             if (a.slopes) sc -= a.slopes[head] * (float)(pos - j);
         }
-        const float m_new = fmaxf(m, warp_max(sc));
-        const float alpha = expf(m - m_new);
-        const float p = valid ? expf(sc - m_new) : 0.f;
-        l = l * alpha + warp_sum(p);
-        m = m_new;
+        float p;
+        if (a.score_bias) {
+            p = valid ? 1.0f / (1.0f + expf(-(sc + a.score_bias[head]))) : 0.f;
+        } else {
+            const float m_new = fmaxf(m, warp_max(sc));
+            const float alpha = expf(m - m_new);
+            p = valid ? expf(sc - m_new) : 0.f;
+            l = l * alpha + warp_sum(p);
+            m = m_new;
 #pragma unroll
-        for (int i = 0; i < IDM_MAX_HEAD_DIM / 32; ++i) acc[i] *= alpha;
+            for (int i = 0; i < IDM_MAX_HEAD_DIM / 32; ++i) acc[i] *= alpha;
+        }
         const unsigned live = __ballot_sync(0xffffffffu, valid);
         for (int jj = 0; jj < 32; ++jj) {
             if (!((live >> jj) & 1u)) continue;
@@ -110,7 +119,7 @@ __global__ void __launch_bounds__(AG_WARPS * 32) attention_generic_kernel(AttnAr
         }
     }
     T* orow = a.out + (size_t)t * a.out_stride + a.out_col + (size_t)head * a.dv;
-    const float inv = 1.0f / l;
+    const float inv = a.score_bias ? 1.0f : 1.0f / l;
     const float* grow = a.gate && !a.gate_per_head ? a.gate + (size_t)t * a.gate_stride + (size_t)head * a.dv : nullptr;
     const float head_gate = a.gate && a.gate_per_head ? 1.0f / (1.0f + expf(-a.gate[(size_t)t * a.gate_stride + head])) : 1.f;
 #pragma unroll
@@ -151,7 +160,7 @@ extern "C" int idm_attention_generic(const void* q, void* out, void* k_pool, voi
     a.token_seq = token_seq; a.positions = positions; a.slots = slots; a.q_start = q_start; a.cu_q = cu_q;
     a.n_tokens = n_tokens; a.n_q = n_q; a.n_kv = n_kv; a.hd = hd; a.scale = scale; a.window = window;
     a.dv = hd; a.sink = nullptr; a.gate = nullptr; a.gate_stride = 0; a.out_stride = n_q * hd; a.out_col = 0; a.out_scale = 1.f;
-    a.slopes = nullptr; a.gate_per_head = 0; a.softcap = 0.f; a.keep_first = 0;
+    a.slopes = nullptr; a.gate_per_head = 0; a.softcap = 0.f; a.keep_first = 0; a.chunk = 0; a.score_bias = nullptr;
     return attention_generic_launch(a, stream);
 }
 
@@ -179,21 +188,22 @@ extern "C" int idm_attention_sink(const void* q, void* out, int out_stride, int 
     a.n_tokens = n_tokens; a.n_q = n_q; a.n_kv = n_kv; a.hd = hd; a.scale = scale; a.window = window;
     a.dv = dv; a.sink = sink; a.gate = gate; a.gate_stride = gate_stride; a.out_stride = out_stride; a.out_col = out_col;
     a.out_scale = out_scale;
-    a.slopes = nullptr; a.gate_per_head = 0; a.softcap = 0.f; a.keep_first = 0;
+    a.slopes = nullptr; a.gate_per_head = 0; a.softcap = 0.f; a.keep_first = 0; a.chunk = 0; a.score_bias = nullptr;
     return attention_generic_launch(a, stream);
 }
 
 // The same walk once more with every option this kernel has: a window over a cache that keeps all keys (ring 0) or
 // a ring, a sink, a slope per head whose product with the distance p - j is taken off the score, a gate that is
 // one number per head (gate_per_head) or one per channel, a cap on the scores and first keys that every query sees
-// (keep_first; not with a ring, which does not keep them).
+// (keep_first; not with a ring, which does not keep them), chunks instead of a window, and sigmoid weights
+// (score_bias; there is no denominator then, so no sink).
 extern "C" int idm_attention_biased(const void* q, void* out, int out_stride, int out_col, float out_scale,
                                     void* k_pool, void* v_pool, const int* table, int table_stride, int ring,
                                     const float* sink, const float* slopes, const float* gate, int gate_stride,
                                     int gate_per_head, const int* token_seq, const int* positions, const int* slots,
                                     const int* q_start, const int* cu_q, int n_tokens, int n_q, int n_kv,
-                                    int hd, int dv, float scale, int window, float softcap, int keep_first,
-                                    cudaStream_t stream) {
+                                    int hd, int dv, float scale, int window, float softcap, int keep_first, int chunk,
+                                    const float* score_bias, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
     IDM_REQUIRE(hd > 0 && hd <= IDM_MAX_HEAD_DIM && dv > 0 && dv <= IDM_MAX_HEAD_DIM,
                 "attention: key and value sizes %d, %d must be at most %d", hd, dv, IDM_MAX_HEAD_DIM);
@@ -202,6 +212,8 @@ extern "C" int idm_attention_biased(const void* q, void* out, int out_stride, in
                 out_col + n_q * dv, out_stride);
     IDM_REQUIRE(keep_first >= 0 && softcap >= 0.f && (keep_first == 0 || ring == 0),
                 "attention: keep_first=%d softcap=%g ring=%d (a ring does not keep a sequence's first keys)", keep_first, softcap, ring);
+    IDM_REQUIRE(chunk >= 0 && (chunk == 0 || (window <= 0 && ring == 0)), "attention: chunks of %d with a window of %d, ring %d", chunk, window, ring);
+    IDM_REQUIRE(score_bias == nullptr || sink == nullptr, "attention: sigmoid weights have no denominator for a sink to join");
     AttnArgs a;
     a.q = (const T*)q; a.out = (T*)out;
     a.cache = KVAddr{(T*)k_pool, (T*)v_pool, table, table_stride, ring, n_kv, hd};
@@ -210,6 +222,6 @@ extern "C" int idm_attention_biased(const void* q, void* out, int out_stride, in
     a.n_tokens = n_tokens; a.n_q = n_q; a.n_kv = n_kv; a.hd = hd; a.scale = scale; a.window = window;
     a.dv = dv; a.sink = sink; a.gate = gate; a.gate_stride = gate_stride; a.out_stride = out_stride; a.out_col = out_col;
     a.out_scale = out_scale; a.slopes = slopes; a.gate_per_head = gate_per_head;
-    a.softcap = softcap; a.keep_first = keep_first;
+    a.softcap = softcap; a.keep_first = keep_first; a.chunk = chunk; a.score_bias = score_bias;
     return attention_generic_launch(a, stream);
 }

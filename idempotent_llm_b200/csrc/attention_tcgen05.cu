@@ -22,6 +22,11 @@
 // block walk a tile's runs and fold as it goes, keeping O in scratch of its own.  Either way a row is the
 // same sequence of operations on the same numbers: the same bits (tests compare them).
 //
+// Chunks (chunk > 0): a query sees the keys of its own chunk of positions only; runs before the first chunk any row of a
+// tile is in are not walked, the rest is masked.  Sigmoid weights (score_bias): p = 1 / (1 + 2^-(s + bias)) for every
+// visible key, no maximum, no sum, nothing divided at the end; a run's (m, l) are (0, 0), which makes every coefficient
+// of the fold exactly 1.
+//
 // Masked keys give p = 0 exactly (select, not arithmetic); a row that sees no key of a run leaves that
 // run out; rows of V past the sequence's length are zeroed in shared memory before they meet the MMA,
 // so stale page contents cannot leak.  Rows of a tile beyond its tokens are not worked on.
@@ -75,6 +80,8 @@ struct AttnTcArgs {
     const float* slopes;                               // [n_q] or null: slopes[head] * (p - j) is taken off the scaled score of key j
     int window;                                        // > 0: a query at p sees keys p - window + 1 .. p; 0: every earlier key
     int keep_first;                                    // > 0 (with a window): keys j < keep_first are seen from any distance
+    int chunk;                                         // > 0 (no window): a query at p sees keys p - p % chunk .. p
+    const float* score_bias;                           // [n_q] or null: weights sigmoid(score + score_bias[head]) instead of a softmax
     float cap_in, cap_out;                             // cap_in > 0: a raw score s becomes cap_out * tanh(s * cap_in), which is
                                                        // (cap / scale) tanh(s scale / cap): the cap on the scaled score, in raw units
     const int* tile_seq; const int* tile_start;
@@ -110,6 +117,19 @@ struct AttnTcSmem {
     // leaves 512 bytes to reach the border (the array is declared with that alignment; the kernel checks)
     static constexpr int TOTAL = NEED + (HD == 128 ? 512 : 1024);
 };
+
+// the first key a query at position p sees, kept first keys aside
+__device__ __forceinline__ int attn_first_seen(const AttnTcArgs& a, int p) {
+    return a.chunk > 0 ? p - p % a.chunk : a.window > 0 ? max(0, p - a.window + 1) : 0;
+}
+// what a row's context is multiplied with at its end
+__device__ __forceinline__ float attn_final_factor(const AttnTcArgs& a, float L) { return a.score_bias ? 1.0f : __fdiv_rn(1.0f, L); }
+// sigmoid(s * scale + bias) of a raw score, with neg_scale = -scale log2(e), neg_bias = -bias log2(e); 0 for -inf
+__device__ __forceinline__ float sigmoid_weight(float s, float neg_scale, float neg_bias) {
+    float r;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(__fadd_rn(1.0f, ex2_hw(__fmaf_rn(s, neg_scale, neg_bias)))));
+    return r;
+}
 
 // One step of the fold of a run's (m, l) into the row's (M, L); a, b: what the contexts are scaled by.
 // A run (or a start) without a key has m = -inf and drops out exactly.
@@ -187,7 +207,7 @@ __device__ __forceinline__ void fold_runs_and_store(const AttnTcArgs& a, const f
             const float sa = fold_sink(a.sink, head0 + (row & (gp - 1)), M, L);
             acc.x = __fmul_rn(acc.x, sa); acc.y = __fmul_rn(acc.y, sa);
         }
-        const float inv = __fdiv_rn(1.0f, L);
+        const float inv = attn_final_factor(a, L);
         T* dst = a.out + ((size_t)(tok0 + (row >> gs)) * a.n_q + head0 + (row & (gp - 1))) * HD + c4 * 4 + 2 * half;
         *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(__fmul_rn(acc.x, inv), __fmul_rn(acc.y, inv));
     }
@@ -239,7 +259,7 @@ __device__ __forceinline__ void fold_rows_and_store(const AttnTcArgs& a, const f
 #pragma unroll
             for (int i = 0; i < 16; ++i) acc[i] = __fmul_rn(acc[i], sa);
         }
-        store_out16(dst + c, acc, __fdiv_rn(1.0f, L));
+        store_out16(dst + c, acc, attn_final_factor(a, L));
     }
 }
 
@@ -267,7 +287,7 @@ __device__ __forceinline__ void count_and_fold_runs(const AttnTcArgs& a, const f
 
 #include "attention_few_rows.cuh"
 
-template <int HD>
+template <int HD, bool SIG>
 __global__ void __launch_bounds__(AP_THREADS, 2)
 attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                     const __grid_constant__ CUtensorMap map_v, AttnTcArgs a) {
@@ -327,7 +347,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     // in walk order, walk_of(run) a run's first block.  A run starts wherever block_of(w) is a multiple of R, which
     // the first block behind the gap is too.
     const int W = a.window;
-    const int win_run = W > 0 ? (max(0, p_first - W + 1) / AP_BN) / R : 0;
+    const int win_run = (attn_first_seen(a, p_first) / AP_BN) / R;
     const int kb = (W > 0 && a.keep_first > 0) ? (min(a.keep_first, p_last + 1) + AP_BN - 1) / AP_BN : 0;
     const bool gap = kb > 0 && kb < win_run * R;                 // (kept blocks that reach the window's first run: one walk from 0)
     const int run_lo = (kb > 0 && !gap) ? 0 : win_run;           // the first run walked behind the kept blocks' own
@@ -453,6 +473,9 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         const bool row_live = r < rows_valid;
         const bool warp_live = warp * 32 < rows_valid;           // (a warp without rows keeps the barriers' count and no more)
         const int p_r = p_first + (r >> gs);
+        const int lo_r = attn_first_seen(a, p_r);                // the first key the row sees, kept ones aside
+        const float neg_scale = -a.scale_log2;
+        const float neg_bias = SIG ? -__fmul_rn(a.score_bias[head0 + (r & (gp - 1))], 1.4426950408889634f) : 0.f;
         // the slope in units of the raw score (the scale is positive): raw + slope_raw * (j - p) is what is scaled
         const float slope_raw = a.slopes ? __fdiv_rn(__fmul_rn(a.slopes[head0 + (r & (gp - 1))], 1.4426950408889634f), a.scale_log2) : 0.f;
         const uint32_t lane_base = (uint32_t)(warp * 32) << 16;
@@ -487,7 +510,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             }
             if (r < cap) reinterpret_cast<float2*>(part0 + (size_t)which * part_floats + (size_t)HD * cap)[r] = make_float2(m_run, l_run);
         };
-        float m_ref = -INFINITY, l = 0.f;                        // the current run
+        constexpr float M_NONE = SIG ? 0.f : -INFINITY;          // where a run's maximum starts
+        float m_ref = M_NONE, l = 0.f;                           // the current run
         float M_tot = -INFINITY, L_tot = 0.f;                    // the runs folded so far
         bool ok = true;
         for (int b = 0; b < nb && ok; ++b) {
@@ -497,7 +521,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             tc_fence_after();
             const bool run_start = b > 0 && block_of(b_first + b) % R == 0;
             float m_prev = 0.f, l_prev = 0.f;
-            if (run_start) { m_prev = m_ref; l_prev = l; m_ref = -INFINITY; l = 0.f; }
+            if (run_start) { m_prev = m_ref; l_prev = l; m_ref = M_NONE; l = 0.f; }
             uint32_t sr[AP_BN];
             if (warp_live) {
                 tc_ld32_issue(tmem + lane_base + (uint32_t)(b & 1) * AP_BN, sr);
@@ -525,10 +549,10 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                     for (int j = 0; j < AP_BN; ++j)
                         if (key0 + j > p_r) sr[j] = 0xff800000u;  // -inf: p becomes 0 exactly
                 }
-                if (W > 0 && key0 + W <= p_r) {                   // some key of the block lies before the row's window
+                if (key0 < lo_r) {                                // some key of the block lies before the row's window or chunk
 #pragma unroll
                     for (int j = 0; j < AP_BN; ++j)
-                        if (key0 + j + W <= p_r && key0 + j >= a.keep_first) sr[j] = 0xff800000u;
+                        if (key0 + j < lo_r && key0 + j >= a.keep_first) sr[j] = 0xff800000u;
                 }
                 if (a.slopes) {
                     const float d0 = (float)(key0 - p_r);
@@ -536,37 +560,46 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                     for (int j = 0; j < AP_BN; ++j)
                         sr[j] = __float_as_uint(__fmaf_rn(slope_raw, d0 + (float)j, __uint_as_float(sr[j])));
                 }
-                // the maximum of the raw scores (the scale is positive), four chains side by side
-                // (the three-input maximum of sm_100: two scores per instruction)
-                float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+                if constexpr (SIG) {
 #pragma unroll
-                for (int j = 0; j < AP_BN; j += 8) {
+                    for (int j = 0; j < AP_BN; j += 2) {
+                        const __nv_bfloat162 pk = __floats2bfloat162_rn(sigmoid_weight(__uint_as_float(sr[j]), neg_scale, neg_bias),
+                                                                        sigmoid_weight(__uint_as_float(sr[j + 1]), neg_scale, neg_bias));
+                        packed[j / 2] = *reinterpret_cast<const uint32_t*>(&pk);
+                    }
+                } else {
+                    // the maximum of the raw scores (the scale is positive), four chains side by side
+                    // (the three-input maximum of sm_100: two scores per instruction)
+                    float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-                    for (int u = 0; u < 4; ++u)
-                        mx[u] = max3(mx[u], __uint_as_float(sr[j + 2 * u]), __uint_as_float(sr[j + 2 * u + 1]));
-                }
-                const float m_blk = __fmul_rn(fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])), a.scale_log2);
-                if (m_blk > m_ref + AP_RESCALE_STEP) {             // (never for a block without a visible key: -inf)
-                    alpha = exp2f(m_ref - m_blk);                  // 0 at a run's first visible key
-                    m_ref = m_blk;
-                }
-                // p = 2^(s * scale - m_ref): one fused multiply-add and one exponential per score; before the
-                // run's first visible key every score is -inf and p = 2^(-inf) = 0
-                const float neg_m = m_ref == -INFINITY ? 0.f : -m_ref;
-                float sum4[4] = {0.f, 0.f, 0.f, 0.f};
+                    for (int j = 0; j < AP_BN; j += 8) {
 #pragma unroll
-                for (int j = 0; j < AP_BN; j += 4) {
-                    const float p0 = ex2_hw(__fmaf_rn(__uint_as_float(sr[j]), a.scale_log2, neg_m));
-                    const float p1 = ex2_hw(__fmaf_rn(__uint_as_float(sr[j + 1]), a.scale_log2, neg_m));
-                    const float p2 = ex2_hw(__fmaf_rn(__uint_as_float(sr[j + 2]), a.scale_log2, neg_m));
-                    const float p3 = ex2_hw(__fmaf_rn(__uint_as_float(sr[j + 3]), a.scale_log2, neg_m));
-                    sum4[0] = __fadd_rn(sum4[0], p0); sum4[1] = __fadd_rn(sum4[1], p1);
-                    sum4[2] = __fadd_rn(sum4[2], p2); sum4[3] = __fadd_rn(sum4[3], p3);
-                    const __nv_bfloat162 pa = __floats2bfloat162_rn(p0, p1), pb = __floats2bfloat162_rn(p2, p3);
-                    packed[j / 2] = *reinterpret_cast<const uint32_t*>(&pa);
-                    packed[j / 2 + 1] = *reinterpret_cast<const uint32_t*>(&pb);
+                        for (int u = 0; u < 4; ++u)
+                            mx[u] = max3(mx[u], __uint_as_float(sr[j + 2 * u]), __uint_as_float(sr[j + 2 * u + 1]));
+                    }
+                    const float m_blk = __fmul_rn(fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])), a.scale_log2);
+                    if (m_blk > m_ref + AP_RESCALE_STEP) {             // (never for a block without a visible key: -inf)
+                        alpha = exp2f(m_ref - m_blk);                  // 0 at a run's first visible key
+                        m_ref = m_blk;
+                    }
+                    // p = 2^(s * scale - m_ref): one fused multiply-add and one exponential per score; before the
+                    // run's first visible key every score is -inf and p = 2^(-inf) = 0
+                    const float neg_m = m_ref == -INFINITY ? 0.f : -m_ref;
+                    float sum4[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+                    for (int j = 0; j < AP_BN; j += 4) {
+                        const float p0 = ex2_hw(__fmaf_rn(__uint_as_float(sr[j]), a.scale_log2, neg_m));
+                        const float p1 = ex2_hw(__fmaf_rn(__uint_as_float(sr[j + 1]), a.scale_log2, neg_m));
+                        const float p2 = ex2_hw(__fmaf_rn(__uint_as_float(sr[j + 2]), a.scale_log2, neg_m));
+                        const float p3 = ex2_hw(__fmaf_rn(__uint_as_float(sr[j + 3]), a.scale_log2, neg_m));
+                        sum4[0] = __fadd_rn(sum4[0], p0); sum4[1] = __fadd_rn(sum4[1], p1);
+                        sum4[2] = __fadd_rn(sum4[2], p2); sum4[3] = __fadd_rn(sum4[3], p3);
+                        const __nv_bfloat162 pa = __floats2bfloat162_rn(p0, p1), pb = __floats2bfloat162_rn(p2, p3);
+                        packed[j / 2] = *reinterpret_cast<const uint32_t*>(&pa);
+                        packed[j / 2 + 1] = *reinterpret_cast<const uint32_t*>(&pb);
+                    }
+                    row_sum = __fadd_rn(__fadd_rn(sum4[0], sum4[1]), __fadd_rn(sum4[2], sum4[3]));
                 }
-                row_sum = __fadd_rn(__fadd_rn(sum4[0], sum4[1]), __fadd_rn(sum4[2], sum4[3]));
             }
             if (b >= 1) {
                 ok = mbar_wait(o_done, (b - 1) & 1, abort_flag, &g_attn_tc_error);   // P is free, O is settled
@@ -670,7 +703,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             const bool first = tot == nullptr;
             fold_coeffs(M_tot, L_tot, m_ref, l, a_, b_);
             const float sa = (a.sink && row_live) ? fold_sink(a.sink, head0 + (r & (gp - 1)), M_tot, L_tot) : 1.0f;
-            const float inv = __fdiv_rn(1.0f, L_tot);
+            const float inv = SIG ? 1.0f : __fdiv_rn(1.0f, L_tot);
             const float4* mine = reinterpret_cast<const float4*>(tot);
 #pragma unroll 1
             for (int c = 0; c < HD; c += 16) {
@@ -699,20 +732,20 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     if (warp == 5) tmem_dealloc(tmem, AP_TMEM_COLS);
 }
 
-template <int HD>
+template <int HD, bool SIG>
 static int launch_attention_tc(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const AttnTcArgs& a,
                                int n_tiles, cudaStream_t stream) {
     using S = AttnTcSmem<HD>;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, S::TOTAL);
+        cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel<HD, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, S::TOTAL);
         IDM_REQUIRE(e == cudaSuccess, "attention_tc: cannot get %d bytes of shared memory: %s", S::TOTAL,
                     cudaGetErrorString(e));
         configured = true;
     }
     const int n_hg = a.n_q >> a.gp_shift;
     dim3 grid(n_hg * (a.max_runs > 0 ? a.max_runs : a.max_parts > 0 ? a.max_parts : 1), n_tiles);
-    idm_launch(attention_tc_kernel<HD>, dim3(grid), dim3(AP_THREADS), S::TOTAL, stream, mq, mk, mv, a);
+    idm_launch(attention_tc_kernel<HD, SIG>, dim3(grid), dim3(AP_THREADS), S::TOTAL, stream, mq, mk, mv, a);
     IDM_LAUNCH_CHECK("attention_tc");
     return 0;
 }
@@ -746,7 +779,7 @@ extern "C" long long idm_attention_tc_scratch_floats(int n_tiles, int n_q, int n
 // block of its own and results meet in scratch; max_runs == 0:
 // one block per tile and head group (`scratch` may be null if no tile has more than run_blocks key blocks).
 static int attention_tc_any(const void* q, void* out, const float* sink, const float* slopes, int window, float softcap, int keep_first,
-                            const void* k_pool, const void* v_pool, int n_pages,
+                            int chunk, const float* score_bias, const void* k_pool, const void* v_pool, int n_pages,
                             const int* table, int table_stride, const int* tile_seq, const int* tile_start,
                             int n_tiles, const int* cu_q, const int* q_start, const int* kv_len,
                             const int* slots, int n_tokens, int n_q, int n_kv, int hd, float scale,
@@ -788,6 +821,7 @@ static int attention_tc_any(const void* q, void* out, const float* sink, const f
     AttnTcArgs a;
     a.out = (T*)out; a.sink = sink; a.slopes = slopes; a.window = window > 0 ? window : 0;
     a.keep_first = (window > 0 && keep_first > 0) ? keep_first : 0;
+    a.chunk = chunk; a.score_bias = score_bias;
     a.cap_in = softcap > 0.f ? scale / softcap : 0.f; a.cap_out = softcap > 0.f ? softcap / scale : 0.f;
     a.tile_seq = tile_seq; a.tile_start = tile_start; a.cu_q = cu_q; a.q_start = q_start;
     a.kv_len = kv_len; a.slots = slots; a.table = table; a.table_stride = table_stride;
@@ -799,11 +833,18 @@ static int attention_tc_any(const void* q, void* out, const float* sink, const f
     IDM_REQUIRE(a.max_parts == 0 || (scratch != nullptr && runs_per_part >= 1 && groups <= AP_COUNTERS),
                 "attention_tc: shared tiles need scratch, runs_per_part >= 1 and at most %d tiles x head groups (got %lld)", AP_COUNTERS, groups);
     // (the kernel for few rows has neither windows nor slopes nor a cap: such layers' single tokens take the general one, a block a run)
-    if (g_attn_few_rows && slopes == nullptr && window <= 0 && !(softcap > 0.f) && attention_few_rows_can(hd, rows_cap, run_blocks, max_runs, groups))
-        return hd == 64 ? launch_attention_few_rows<64>(mk, mv, a, (const T*)q, n_tiles, stream)
-                        : launch_attention_few_rows<128>(mk, mv, a, (const T*)q, n_tiles, stream);
-    return hd == 64 ? launch_attention_tc<64>(mq, mk, mv, a, n_tiles, stream)
-                    : launch_attention_tc<128>(mq, mk, mv, a, n_tiles, stream);
+    if (g_attn_few_rows && slopes == nullptr && window <= 0 && !(softcap > 0.f) && attention_few_rows_can(hd, rows_cap, run_blocks, max_runs, groups)) {
+        if (score_bias) return hd == 64 ? launch_attention_few_rows<64, AF_SIGMOID>(mk, mv, a, (const T*)q, n_tiles, stream)
+                                        : launch_attention_few_rows<128, AF_SIGMOID>(mk, mv, a, (const T*)q, n_tiles, stream);
+        if (chunk > 0) return hd == 64 ? launch_attention_few_rows<64, AF_CHUNK>(mk, mv, a, (const T*)q, n_tiles, stream)
+                                       : launch_attention_few_rows<128, AF_CHUNK>(mk, mv, a, (const T*)q, n_tiles, stream);
+        return hd == 64 ? launch_attention_few_rows<64, AF_PLAIN>(mk, mv, a, (const T*)q, n_tiles, stream)
+                        : launch_attention_few_rows<128, AF_PLAIN>(mk, mv, a, (const T*)q, n_tiles, stream);
+    }
+    if (score_bias) return hd == 64 ? launch_attention_tc<64, true>(mq, mk, mv, a, n_tiles, stream)
+                                    : launch_attention_tc<128, true>(mq, mk, mv, a, n_tiles, stream);
+    return hd == 64 ? launch_attention_tc<64, false>(mq, mk, mv, a, n_tiles, stream)
+                    : launch_attention_tc<128, false>(mq, mk, mv, a, n_tiles, stream);
 }
 
 extern "C" int idm_attention_tc(const void* q, void* out, const void* k_pool, const void* v_pool, int n_pages,
@@ -812,7 +853,7 @@ extern "C" int idm_attention_tc(const void* q, void* out, const void* k_pool, co
                                 const int* slots, int n_tokens, int n_q, int n_kv, int hd, float scale,
                                 int run_blocks, int max_runs, int rows_cap, float* scratch, const int* tile_pool,
                                 int max_parts, int runs_per_part, cudaStream_t stream) {
-    return attention_tc_any(q, out, nullptr, nullptr, 0, 0.f, 0, k_pool, v_pool, n_pages, table, table_stride, tile_seq, tile_start, n_tiles, cu_q,
+    return attention_tc_any(q, out, nullptr, nullptr, 0, 0.f, 0, 0, nullptr, k_pool, v_pool, n_pages, table, table_stride, tile_seq, tile_start, n_tiles, cu_q,
                             q_start, kv_len, slots, n_tokens, n_q, n_kv, hd, scale, run_blocks, max_runs, rows_cap, scratch,
                             tile_pool, max_parts, runs_per_part, stream);
 }
@@ -825,7 +866,7 @@ extern "C" int idm_attention_tc_sink(const void* q, void* out, const float* sink
                                      const int* kv_len, const int* slots, int n_tokens, int n_q, int n_kv, int hd,
                                      float scale, int run_blocks, int max_runs, int rows_cap, float* scratch,
                                      const int* tile_pool, int max_parts, int runs_per_part, cudaStream_t stream) {
-    return attention_tc_any(q, out, sink, nullptr, 0, 0.f, 0, k_pool, v_pool, n_pages, table, table_stride, tile_seq, tile_start, n_tiles, cu_q,
+    return attention_tc_any(q, out, sink, nullptr, 0, 0.f, 0, 0, nullptr, k_pool, v_pool, n_pages, table, table_stride, tile_seq, tile_start, n_tiles, cu_q,
                             q_start, kv_len, slots, n_tokens, n_q, n_kv, hd, scale, run_blocks, max_runs, rows_cap, scratch,
                             tile_pool, max_parts, runs_per_part, stream);
 }
@@ -834,9 +875,11 @@ extern "C" int idm_attention_tc_sink(const void* q, void* out, const float* sink
 // the distance to a key is taken off its scaled score), a window (> 0: a query sees itself and the window - 1 keys
 // before it; the cache keeps every key, runs of key blocks that no row of a tile sees are not walked), first keys that
 // stay seen behind the window (keep_first), and a cap on the scaled scores (softcap > 0: cap * tanh(score / cap), by
-// the hardware's tanh, whose error is below the rounding of the softmax's weights to bfloat16).
+// the hardware's tanh, whose error is below the rounding of the softmax's weights to bfloat16); or chunks instead of a
+// window (chunk > 0), and sigmoid weights instead of a softmax (score_bias: a number per q-head added to the scaled score).
 extern "C" int idm_attention_tc_biased(const void* q, void* out, const float* sink, const float* slopes, int window,
-                                       float softcap, int keep_first, const void* k_pool, const void* v_pool, int n_pages, const int* table,
+                                       float softcap, int keep_first, int chunk, const float* score_bias,
+                                       const void* k_pool, const void* v_pool, int n_pages, const int* table,
                                        int table_stride, const int* tile_seq, const int* tile_start, int n_tiles,
                                        const int* cu_q, const int* q_start, const int* kv_len, const int* slots,
                                        int n_tokens, int n_q, int n_kv, int hd, float scale, int run_blocks, int max_runs,
@@ -844,7 +887,9 @@ extern "C" int idm_attention_tc_biased(const void* q, void* out, const float* si
                                        int runs_per_part, cudaStream_t stream) {
     IDM_REQUIRE(scale > 0.f, "attention_tc: the scale of the scores must be positive, not %g", (double)scale);
     IDM_REQUIRE(keep_first >= 0 && softcap >= 0.f, "attention_tc: keep_first=%d softcap=%g", keep_first, (double)softcap);
-    return attention_tc_any(q, out, sink, slopes, window, softcap, keep_first, k_pool, v_pool, n_pages, table, table_stride, tile_seq, tile_start,
+    IDM_REQUIRE(chunk >= 0 && (chunk == 0 || window <= 0), "attention_tc: chunks of %d with a window of %d", chunk, window);
+    IDM_REQUIRE(score_bias == nullptr || sink == nullptr, "attention_tc: sigmoid weights have no denominator for a sink to join");
+    return attention_tc_any(q, out, sink, slopes, window, softcap, keep_first, chunk, score_bias, k_pool, v_pool, n_pages, table, table_stride, tile_seq, tile_start,
                             n_tiles, cu_q, q_start, kv_len, slots, n_tokens, n_q, n_kv, hd, scale, run_blocks, max_runs,
                             rows_cap, scratch, tile_pool, max_parts, runs_per_part, stream);
 }

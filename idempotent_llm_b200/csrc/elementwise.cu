@@ -623,19 +623,22 @@ extern "C" int idm_post_pre_norm(float* h, const float* y, const float* w_post, 
 // (gated_act in common.cuh: act 0 is g * sigmoid(g) * u, act 1 the tanh form of gelu times u)
 
 // y[t, i] = act(gu[t, i]) * gu[t, inter + i] of a 32-bit gate/up product [N, 2 * inter]
-__global__ void __launch_bounds__(256) gated_act_kernel(const float* __restrict__ gu, T* __restrict__ y, int inter, int act) {
+__global__ void __launch_bounds__(256) gated_act_kernel(const float* __restrict__ gu, T* __restrict__ y, int inter, int act,
+                                                        const float* __restrict__ row_w) {
     pdl_launch_dependents();
     pdl_wait();
     const int c = blockIdx.y * blockDim.x + threadIdx.x;
     if (c >= inter) return;
     const size_t t = blockIdx.x;
-    from_f32(y[t * (size_t)inter + c], gated_act(gu[t * 2 * (size_t)inter + c], gu[t * 2 * (size_t)inter + inter + c], act));
+    float g = gu[t * 2 * (size_t)inter + c], u = gu[t * 2 * (size_t)inter + inter + c];
+    if (row_w) { g *= row_w[t]; u *= row_w[t]; }                 // a factor on the row's input (gate and up are linear)
+    from_f32(y[t * (size_t)inter + c], gated_act(g, u, act));
 }
 
-extern "C" int idm_gated_act(const float* gu, void* y, int n_tokens, int inter, int act, cudaStream_t stream) {
+extern "C" int idm_gated_act(const float* gu, void* y, int n_tokens, int inter, int act, const float* row_w, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
     IDM_REQUIRE(inter > 0 && act >= 0 && act <= 2, "gated_act: inter=%d act=%d", inter, act);
-    idm_launch(gated_act_kernel, dim3(n_tokens, (inter + 255) / 256), dim3(256), 0, stream, gu, (T*)y, inter, act);
+    idm_launch(gated_act_kernel, dim3(n_tokens, (inter + 255) / 256), dim3(256), 0, stream, gu, (T*)y, inter, act, row_w);
     IDM_LAUNCH_CHECK("gated_act");
     return 0;
 }

@@ -9,8 +9,15 @@
 // step's choices [rows, top], and `pair_w` [rows, top] (null: 1) is the weight of every (token, choice) beside the
 // constant `weight`.  Where an expert's activations are 32-bit numbers of these kernels' own, the pair's weight is
 // multiplied into them (the down product is linear); where the library's products make them, the weight is applied
-// when the experts' outputs are added.
+// when the experts' outputs are added.  With `weight_in` the pair's weight belongs on the expert's INPUT instead: gate and
+// up are linear, so both of a pair's pre-activations are multiplied by it, in 32-bit, wherever they are made, and the
+// outputs are added as they are.
 #include "common.cuh"
+
+// a pair's activation: the weight on what the activation gives, or (weight_in) on both of its arguments
+__device__ __forceinline__ float pair_act(float g, float u, float pw, int weight_in, int act) {
+    return weight_in ? gated_act(g * pw, u * pw, act) : gated_act(g, u, act) * pw;
+}
 
 __device__ __forceinline__ float row_dot(const T* __restrict__ w, const float* __restrict__ xs, int K, int lane, bool vec) {
     float s = 0.f;
@@ -76,7 +83,7 @@ __global__ void __launch_bounds__(256) experts_gate_up_kernel(const T* __restric
                                                               const T* __restrict__ gate_up, long long expert_stride,
                                                               long long row_stride, long long up_off,
                                                               float* __restrict__ a, int width, int ff, int top, int n_experts,
-                                                              int act) {
+                                                              int act, int weight_in) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ float xs[];
@@ -93,7 +100,7 @@ __global__ void __launch_bounds__(256) experts_gate_up_kernel(const T* __restric
         const T* row = gate_up + (size_t)e * expert_stride + (size_t)f * row_stride;
         float g, u;
         row_dot2(row, row + up_off, xs, xs, width, lane, vec, g, u);
-        if (lane == 0) a[(size_t)tk * ff + f] = pair_w ? gated_act(g, u, act) * pw : gated_act(g, u, act);
+        if (lane == 0) a[(size_t)tk * ff + f] = pair_w ? pair_act(g, u, pw, weight_in, act) : gated_act(g, u, act);
     }
 }
 
@@ -138,7 +145,7 @@ __global__ void __launch_bounds__(256) experts_down_kernel(const float* __restri
 extern "C" int idm_experts_few(const void* x, const int* tokens, const int* table, const float* pair_w, const void* gate_up, long long expert_stride,
                                long long row_stride, long long up_off, const void* down,
                                float* a, float* h, int n_tokens, int width, int ff, int top, int n_experts, int act,
-                               float weight, cudaStream_t stream) {
+                               float weight, int weight_in, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
     IDM_REQUIRE(width > 0 && ff > 0 && top > 0 && n_experts > 0 && (act >= 0 && act <= 2), "experts: width=%d ff=%d top=%d experts=%d act=%d",
                 width, ff, top, n_experts, act);
@@ -151,7 +158,7 @@ extern "C" int idm_experts_few(const void* x, const int* tokens, const int* tabl
     const int by1 = max(1, min((ff + 7) / 8, 592 / max(1, n_tokens * top)));
     const int by2 = max(1, min((width + 7) / 8, 592 / max(1, n_tokens)));
     idm_launch(experts_gate_up_kernel, dim3(n_tokens * top, by1), dim3(256), s1, stream, (const T*)x, tokens, table, pair_w, (const T*)gate_up,
-               expert_stride, row_stride, up_off, a, width, ff, top, n_experts, act);
+               expert_stride, row_stride, up_off, a, width, ff, top, n_experts, act, weight_in);
     IDM_LAUNCH_CHECK("experts_gate_up");
     idm_launch(experts_down_kernel, dim3(n_tokens, by2), dim3(256), s2, stream, (const float*)a, tokens, table, (const T*)down, h, width,
                ff, top, n_experts, weight);
@@ -200,6 +207,22 @@ extern "C" int idm_experts_combine(const float* z, const int* place, const float
     return 0;
 }
 
+// out[place[p]] = pair_w[p] for every (token, choice) p that has a grouped row
+__global__ void __launch_bounds__(256) rows_weight_kernel(const float* __restrict__ pair_w, const int* __restrict__ place,
+                                                          float* __restrict__ out, int n_pairs) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int p = blockIdx.x * blockDim.x + threadIdx.x;
+    if (p < n_pairs && place[p] >= 0) out[place[p]] = pair_w[p];
+}
+
+extern "C" int idm_rows_weight(const float* pair_w, const int* place, float* out, int n_pairs, cudaStream_t stream) {
+    if (n_pairs == 0) return 0;
+    idm_launch(rows_weight_kernel, dim3((n_pairs + 255) / 256), dim3(256), 0, stream, pair_w, place, out, n_pairs);
+    IDM_LAUNCH_CHECK("rows_weight");
+    return 0;
+}
+
 // ------------------------------------------------------------------ the same, expert by expert
 // For steps of more than a few tokens whose ids exist on the device only: a block has one expert and a slice of its
 // rows, finds the (token, choice) pairs that use the expert (in ascending order), and walks them eight at a time: the
@@ -214,7 +237,7 @@ __global__ void __launch_bounds__(256) experts_major_kernel(const T* __restrict_
                                                             const float* __restrict__ pair_w,
                                                             const T* __restrict__ w, long long expert_stride, long long row_stride,
                                                             long long up_off, float* __restrict__ out, int n_tokens, int top,
-                                                            int K, int rows, int act) {
+                                                            int K, int rows, int act, int weight_in) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ float sm[];
@@ -309,7 +332,7 @@ __global__ void __launch_bounds__(256) experts_major_kernel(const T* __restrict_
                 for (int tt = 0; tt < EX_TOKENS; ++tt)
                     if (tt < np) {
                         const int pr = pairs[p0 + tt];
-                        out[(size_t)pr * rows + r] = MODE == 0 ? (pair_w ? gated_act(g[tt], u[tt], act) * pair_w[pr] : gated_act(g[tt], u[tt], act)) : g[tt];
+                        out[(size_t)pr * rows + r] = MODE == 0 ? (pair_w ? pair_act(g[tt], u[tt], pair_w[pr], weight_in, act) : gated_act(g[tt], u[tt], act)) : g[tt];
                     }
             }
         }
@@ -320,7 +343,7 @@ __global__ void __launch_bounds__(256) experts_major_kernel(const T* __restrict_
 extern "C" int idm_experts_major(const void* x, const int* tokens, const int* table, const float* pair_w, const void* gate_up,
                                  long long expert_stride, long long row_stride, long long up_off, const void* down,
                                  float* a, float* z, float* h, int n_tokens, int width, int ff, int top, int n_experts,
-                                 int act, float weight, cudaStream_t stream) {
+                                 int act, float weight, int weight_in, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
     IDM_REQUIRE(width > 0 && ff > 0 && top > 0 && n_experts > 0 && (act >= 0 && act <= 2), "experts: width=%d ff=%d top=%d experts=%d act=%d",
                 width, ff, top, n_experts, act);
@@ -330,10 +353,10 @@ extern "C" int idm_experts_major(const void* x, const int* tokens, const int* ta
     if (s2 > 48 * 1024) cudaFuncSetAttribute(experts_major_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2);
     const int by1 = max(1, min((ff + 7) / 8, 592 / n_experts)), by2 = max(1, min((width + 7) / 8, 592 / n_experts));
     idm_launch(experts_major_kernel<0>, dim3(n_experts, by1), dim3(256), s1, stream, (const T*)x, (const float*)nullptr, tokens, table, pair_w,
-               (const T*)gate_up, expert_stride, row_stride, up_off, a, n_tokens, top, width, ff, act);
+               (const T*)gate_up, expert_stride, row_stride, up_off, a, n_tokens, top, width, ff, act, weight_in);
     IDM_LAUNCH_CHECK("experts_major gate/up");
     idm_launch(experts_major_kernel<1>, dim3(n_experts, by2), dim3(256), s2, stream, (const T*)nullptr, (const float*)a, tokens, table, (const float*)nullptr,
-               (const T*)down, (long long)width * ff, (long long)ff, 0LL, z, n_tokens, top, ff, width, act);
+               (const T*)down, (long long)width * ff, (long long)ff, 0LL, z, n_tokens, top, ff, width, act, 0);
     IDM_LAUNCH_CHECK("experts_major down");
     idm_launch(experts_combine_kernel, dim3(n_tokens), dim3(256), 0, stream, (const float*)z, (const int*)nullptr, (const float*)nullptr, h,
                width, top, weight);
@@ -345,10 +368,11 @@ extern "C" int idm_experts_major(const void* x, const int* tokens, const int* ta
 // Every expert's gated feed-forward over its slice of rows grouped by expert: the library's own matrix products (the
 // gate/up product with the activation as its epilogue, then the down product), expert after expert, from one call.
 // counts: on the HOST, rows of each expert; gate_up [E, tiles * 128, width] alternating rows; down [E, width, ff].
-extern "C" int idm_gemm_bf16_gated(const void* x, const void* w, void* y, int M, int inter, int K, int act, cudaStream_t stream);
+// row_w (or null): a number per grouped row that multiplies the row's pre-activations (a weight on the expert's input).
+extern "C" int idm_gemm_bf16_gated_rows(const void* x, const void* w, void* y, int M, int inter, int K, int act, const float* row_w, cudaStream_t stream);
 extern "C" int idm_gemm_bf16(const void* x, const void* w, float* out, int M, int N, int K, cudaStream_t stream);
 
-extern "C" int idm_experts_grouped(const void* xg, const int* counts, int n_experts, const void* gate_up,
+static int experts_grouped(const void* xg, const float* row_w, const int* counts, int n_experts, const void* gate_up,
                                    long long gate_up_stride, const void* down, long long down_stride, void* y, float* z,
                                    int width, int ff, int act, cudaStream_t stream) {
     IDM_REQUIRE(width > 0 && ff > 0 && width % 8 == 0 && ff % 8 == 0, "experts_grouped: width=%d ff=%d (multiples of 8)", width, ff);
@@ -358,24 +382,33 @@ extern "C" int idm_experts_grouped(const void* xg, const int* counts, int n_expe
         if (c <= 0) continue;
         const T* xe = (const T*)xg + at * width;
         T* ye = (T*)y + at * ff;
-        if (idm_gemm_bf16_gated(xe, (const T*)gate_up + (long long)e * gate_up_stride, ye, c, ff, width, act, stream)) return 1;
+        if (idm_gemm_bf16_gated_rows(xe, (const T*)gate_up + (long long)e * gate_up_stride, ye, c, ff, width, act, row_w ? row_w + at : nullptr, stream)) return 1;
         if (idm_gemm_bf16(ye, (const T*)down + (long long)e * down_stride, z + at * width, c, width, ff, stream)) return 1;
         at += c;
     }
     return 0;
 }
 
+extern "C" int idm_experts_grouped(const void* xg, const int* counts, int n_experts, const void* gate_up,
+                                   long long gate_up_stride, const void* down, long long down_stride, void* y, float* z,
+                                   int width, int ff, int act, cudaStream_t stream) {
+    return experts_grouped(xg, nullptr, counts, n_experts, gate_up, gate_up_stride, down, down_stride, y, z, width, ff, act, stream);
+}
+
 // The grouped feed-forward of a step from one call: rows gathered in the order of their experts (src: grouped row ->
 // token), every expert's two products, outputs added into the stream in the order of a token's choices (place:
-// (token, choice) -> grouped row).  xg, y, z: scratch [n_tokens * top, width | ff | width].
+// (token, choice) -> grouped row).  xg, y, z: scratch [n_tokens * top, width | ff | width].  row_w (scratch [n_tokens *
+// top], or null): the pairs' weights belong on the experts' inputs; they are put in the order of the grouped rows there.
 extern "C" int idm_experts_grouped_step(const void* x, const int* src, const int* place, const float* pair_w, const int* counts, int n_experts,
                                         const void* gate_up, long long gate_up_stride, const void* down, long long down_stride,
                                         void* xg, void* y, float* z, float* h, int n_tokens, int top, int width, int ff, int act,
-                                        float weight, cudaStream_t stream) {
+                                        float weight, float* row_w, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
+    IDM_REQUIRE(row_w == nullptr || pair_w != nullptr, "experts_grouped_step: weights on the inputs need the pairs' weights");
     if (idm_rows_gather(x, src, xg, n_tokens * top, width, stream)) return 1;
-    if (idm_experts_grouped(xg, counts, n_experts, gate_up, gate_up_stride, down, down_stride, y, z, width, ff, act, stream)) return 1;
-    return idm_experts_combine(z, place, pair_w, h, n_tokens, width, top, weight, stream);
+    if (row_w && idm_rows_weight(pair_w, place, row_w, n_tokens * top, stream)) return 1;
+    if (experts_grouped(xg, row_w, counts, n_experts, gate_up, gate_up_stride, down, down_stride, y, z, width, ff, act, stream)) return 1;
+    return idm_experts_combine(z, place, row_w ? nullptr : pair_w, h, n_tokens, width, top, weight, stream);
 }
 
 // Single-token steps of many sequences, whose ids exist on the device only and whose shapes must not change from
@@ -402,17 +435,41 @@ __global__ void __launch_bounds__(256) experts_pick_kernel(const float* __restri
     }
 }
 
+// out[e, t] = the weight of token t's pair that names expert e (0 where none does): one thread per (expert, token)
+__global__ void __launch_bounds__(256) experts_weight_table_kernel(const int* __restrict__ tokens, const int* __restrict__ table,
+                                                                   const float* __restrict__ pair_w, float* __restrict__ out,
+                                                                   int n_tokens, int top, int n_experts) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n_tokens * n_experts) return;
+    const int e = i / n_tokens, t = i % n_tokens;
+    float w = 0.f;
+    for (int k = 0; k < top; ++k)
+        if (table[(size_t)tokens[t] * top + k] == e) w = pair_w[t * top + k];
+    out[i] = w;
+}
+
+// weights_in (scratch [E, n_tokens], or null): the pairs' weights belong on the experts' inputs
 extern "C" int idm_experts_dense(const void* x, const int* tokens, const int* table, const float* pair_w, int n_experts, const void* gate_up,
                                  long long gate_up_stride, const void* down, long long down_stride, void* y, float* z_all,
-                                 float* h, int n_tokens, int width, int ff, int top, int act, float weight, cudaStream_t stream) {
+                                 float* h, int n_tokens, int width, int ff, int top, int act, float weight, float* weights_in,
+                                 cudaStream_t stream) {
     if (n_tokens == 0) return 0;
+    IDM_REQUIRE(weights_in == nullptr || pair_w != nullptr, "experts_dense: weights on the inputs need the pairs' weights");
+    if (weights_in) {
+        idm_launch(experts_weight_table_kernel, dim3((n_tokens * n_experts + 255) / 256), dim3(256), 0, stream, tokens, table, pair_w, weights_in,
+                   n_tokens, top, n_experts);
+        IDM_LAUNCH_CHECK("experts_weight_table");
+    }
     IDM_REQUIRE(width > 0 && ff > 0 && width % 8 == 0 && ff % 8 == 0, "experts_dense: width=%d ff=%d (multiples of 8)", width, ff);
     for (int e = 0; e < n_experts; ++e) {
-        if (idm_gemm_bf16_gated(x, (const T*)gate_up + (long long)e * gate_up_stride, y, n_tokens, ff, width, act, stream)) return 1;
+        if (idm_gemm_bf16_gated_rows(x, (const T*)gate_up + (long long)e * gate_up_stride, y, n_tokens, ff, width, act,
+                                     weights_in ? weights_in + (size_t)e * n_tokens : nullptr, stream)) return 1;
         if (idm_gemm_bf16(y, (const T*)down + (long long)e * down_stride, z_all + (size_t)e * n_tokens * width, n_tokens, width, ff, stream)) return 1;
     }
-    idm_launch(experts_pick_kernel, dim3(n_tokens), dim3(256), 0, stream, (const float*)z_all, tokens, table, pair_w, h, n_tokens, width, top,
-               n_experts, weight);
+    idm_launch(experts_pick_kernel, dim3(n_tokens), dim3(256), 0, stream, (const float*)z_all, tokens, table, weights_in ? (const float*)nullptr : pair_w, h,
+               n_tokens, width, top, n_experts, weight);
     IDM_LAUNCH_CHECK("experts_pick");
     return 0;
 }

@@ -99,6 +99,7 @@ struct GemmEpi {
     float* out;          // STORE: [M, N]; RESIDUAL: the residual stream [M, N]
     T* y; int inter;     // SWIGLU: y [M, inter]
     int act;             // SWIGLU: which gated activation (gated_act in common.cuh; 0 = silu)
+    const float* row_w;  // SWIGLU, or null: row_w[t] multiplies gate and up of token t before the activation
     QkvArgs q;           // QKV
 };
 
@@ -192,7 +193,12 @@ __device__ __forceinline__ void persistent_tile_epilogue(const GemmEpi& e, uint3
                 const int j = fl >> 3, sub = fl & 7;
                 if (j < cols) {
                     const float4* src = reinterpret_cast<const float4*>(xs + j * GT_BM + sub * 16);
-                    const float4 p0 = src[0], p1 = src[1], p2 = src[2], p3 = src[3];
+                    float4 p0 = src[0], p1 = src[1], p2 = src[2], p3 = src[3];
+                    if (e.row_w) {
+                        const float rw = e.row_w[t0 + c0 + j];
+                        p0.x *= rw; p0.y *= rw; p0.z *= rw; p0.w *= rw; p1.x *= rw; p1.y *= rw; p1.z *= rw; p1.w *= rw;
+                        p2.x *= rw; p2.y *= rw; p2.z *= rw; p2.w *= rw; p3.x *= rw; p3.y *= rw; p3.z *= rw; p3.w *= rw;
+                    }
                     const float y8[8] = {gated_act(p0.x, p0.y, e.act), gated_act(p0.z, p0.w, e.act), gated_act(p1.x, p1.y, e.act), gated_act(p1.z, p1.w, e.act),
                                          gated_act(p2.x, p2.y, e.act), gated_act(p2.z, p2.w, e.act), gated_act(p3.x, p3.y, e.act), gated_act(p3.z, p3.w, e.act)};
                     const int fg = tx * 64 + sub * 8;
@@ -1038,6 +1044,7 @@ __global__ void __launch_bounds__(GS_THREADS) gemm_small_kernel(const __grid_con
                 } else if (EPI == EPI_SWIGLU) {
                     // the tile's columns are gate, up, gate, up, ... of the features f0 / 2 ..; 32 columns are asked
                     // for before the first is waited for
+                    const float rw = e.row_w && live ? e.row_w[t] : 1.0f;      // (a factor of 1 changes no bit)
 #pragma unroll 1
                     for (int c0 = 0; c0 < bf; c0 += 32) {
                         if (((f0 + c0) >> 1) >= e.inter) break;
@@ -1053,7 +1060,7 @@ __global__ void __launch_bounds__(GS_THREADS) gemm_small_kernel(const __grid_con
                             float y8[8];
 #pragma unroll
                             for (int i = 0; i < 8; ++i)
-                                y8[i] = gated_act(__uint_as_float(raw[16 * h + 2 * i]), __uint_as_float(raw[16 * h + 2 * i + 1]), e.act);
+                                y8[i] = gated_act(__fmul_rn(__uint_as_float(raw[16 * h + 2 * i]), rw), __fmul_rn(__uint_as_float(raw[16 * h + 2 * i + 1]), rw), e.act);
                             T* dst = e.y + (size_t)t * e.inter + fg;
                             if ((e.inter & 7) == 0 && fg + 8 <= e.inter) {
                                 store8(dst, y8);
@@ -1444,13 +1451,19 @@ extern "C" int idm_gemm_bf16_swiglu(const void* x, const void* w_tiled, void* y,
 }
 
 // the same product with the gated activation chosen by number (gated_act in common.cuh): y = act(x . gate^T) * (x . up^T)
-extern "C" int idm_gemm_bf16_gated(const void* x, const void* w_tiled, void* y, int M, int inter, int K, int act,
-                                   cudaStream_t stream) {
+// with, if given, a factor per row: y[t] = act(row_w[t] x_t . gate^T) * (row_w[t] x_t . up^T)
+extern "C" int idm_gemm_bf16_gated_rows(const void* x, const void* w_tiled, void* y, int M, int inter, int K, int act,
+                                        const float* row_w, cudaStream_t stream) {
     IDM_REQUIRE(act >= 0 && act <= 2, "gemm_gated: activation %d is not built", act);
     GemmEpi e = {};
-    e.y = (T*)y; e.inter = inter; e.act = act;
+    e.y = (T*)y; e.inter = inter; e.act = act; e.row_w = row_w;
     const int tiles = (inter + 63) / 64;
     return gemm_any<EPI_SWIGLU>(x, w_tiled, e, M, tiles * GT_BM, K, stream);
+}
+
+extern "C" int idm_gemm_bf16_gated(const void* x, const void* w_tiled, void* y, int M, int inter, int K, int act,
+                                   cudaStream_t stream) {
+    return idm_gemm_bf16_gated_rows(x, w_tiled, y, M, inter, K, act, nullptr, stream);
 }
 
 // The fused q/k/v projection with the per-head finish (norm, rotation, q out, cache write); head_dim 32, 64 or 128

@@ -10,16 +10,28 @@
 // cache is read once per token and step whatever the number of heads.  All arithmetic here is 32-bit; the cache
 // rows and the value maps' outputs are in the storage type.
 //
-// Rotation: neighbours (2i, 2i+1) of the rotated part are turned by the token's angle i, (u, v) ->
-// (u cos - v sin, v cos + u sin), cos and sin from the step's table times a constant magnitude.
+// Rotation: neighbours (2i, 2i+1) of the rotated part, or (halves) dims i and i + rot_dims / 2, are turned by the token's
+// angle i, (u, v) -> (u cos - v sin, v cos + u sin), cos and sin from the step's table times a constant magnitude.
 #include "common.cuh"
+
+// element d of a rotated part x whose first rot_dims elements are turned; cs: the token's row of the table
+__device__ __forceinline__ float latent_turned(const float* __restrict__ x, int d, int rot_dims, int halves,
+                                               const float2* __restrict__ cs, float mag) {
+    if (d >= rot_dims) return x[d];
+    const int h = rot_dims >> 1;
+    const bool first = halves ? d < h : (d & 1) == 0;
+    const int i = halves ? (first ? d : d - h) : d >> 1, other = halves ? (first ? d + h : d - h) : d ^ 1;
+    const float2 a = cs[i];
+    const float co = a.x * mag, si = a.y * mag;
+    return first ? x[d] * co - x[other] * si : x[d] * co + x[other] * si;
+}
 
 // ------------------------------------------------------------------ the row a token keeps
 // proj [N, ld] 32-bit, columns col0 .. col0 + R: the latent before its norm; the next dr: the shared key part.
 // One block per token: c = x / sqrt(mean(x^2) + eps) * w, r turned; [c | r] to the token's place in the paged
 // pool [pages, PAGE, R + dr] and, if asked for, to packed rows row_out [N, R + dr] (the step's own keys).
 __global__ void __launch_bounds__(128) latent_kv_finish_kernel(const float* __restrict__ proj, int ld, int col0, int R, int dr,
-                                                               int rot_dims, const float* __restrict__ w, float eps,
+                                                               int rot_dims, int halves, const float* __restrict__ w, float eps,
                                                                const float2* __restrict__ cs, int half, float mag,
                                                                T* __restrict__ pool, const int* __restrict__ table,
                                                                int table_stride, const int* __restrict__ token_seq,
@@ -43,24 +55,14 @@ __global__ void __launch_bounds__(128) latent_kv_finish_kernel(const float* __re
         if (row2) from_f32(row2[d], c);
     }
     const float* xr = x + R;
-    for (int i = threadIdx.x; 2 * i < dr; i += blockDim.x) {
-        float u = xr[2 * i], v = (2 * i + 1 < dr) ? xr[2 * i + 1] : 0.f;
-        if (2 * i + 1 < rot_dims) {
-            const float2 a = cs[(size_t)t * half + i];
-            const float co = a.x * mag, si = a.y * mag;
-            const float u2 = u * co - v * si, v2 = v * co + u * si;
-            u = u2; v = v2;
-        }
-        from_f32(row[R + 2 * i], u);
-        if (row2) from_f32(row2[R + 2 * i], u);
-        if (2 * i + 1 < dr) {
-            from_f32(row[R + 2 * i + 1], v);
-            if (row2) from_f32(row2[R + 2 * i + 1], v);
-        }
+    for (int d = threadIdx.x; d < dr; d += blockDim.x) {
+        const float v = latent_turned(xr, d, rot_dims, halves, cs + (size_t)t * half, mag);
+        from_f32(row[R + d], v);
+        if (row2) from_f32(row2[R + d], v);
     }
 }
 
-extern "C" int idm_latent_kv_finish(const float* proj, int ld, int col0, int R, int dr, int rot_dims, const float* w,
+extern "C" int idm_latent_kv_finish(const float* proj, int ld, int col0, int R, int dr, int rot_dims, int halves, const float* w,
                                     float eps, const float* cs, int half, float mag, void* pool, const int* table,
                                     int table_stride, const int* token_seq, const int* positions, const int* slots,
                                     void* row_out, int n_tokens, cudaStream_t stream) {
@@ -68,7 +70,7 @@ extern "C" int idm_latent_kv_finish(const float* proj, int ld, int col0, int R, 
     IDM_REQUIRE(R > 0 && dr >= 0 && col0 >= 0 && col0 + R + dr <= ld, "latent_kv_finish: columns %d + %d + %d of %d", col0, R, dr, ld);
     IDM_REQUIRE(rot_dims >= 0 && rot_dims <= dr && rot_dims % 2 == 0 && (rot_dims == 0 || (cs != nullptr && half >= rot_dims / 2)),
                 "latent_kv_finish: %d turned dims of %d with a table of %d angles", rot_dims, dr, half);
-    idm_launch(latent_kv_finish_kernel, dim3(n_tokens), dim3(128), 0, stream, proj, ld, col0, R, dr, rot_dims, w, eps,
+    idm_launch(latent_kv_finish_kernel, dim3(n_tokens), dim3(128), 0, stream, proj, ld, col0, R, dr, rot_dims, halves, w, eps,
                (const float2*)cs, half, mag, (T*)pool, table, table_stride, token_seq, positions, slots, (T*)row_out);
     IDM_LAUNCH_CHECK("latent_kv_finish");
     return 0;
@@ -88,7 +90,7 @@ static_assert(HW_WARPS == HW_TOKENS, "a warp per token in the last phase");
 template <typename OutT>
 __global__ void __launch_bounds__(HW_WARPS * 32) headwise_kernel(const float* __restrict__ x, long long x_tok, int x_head, int I,
                                                                  const T* __restrict__ W, int O, OutT* __restrict__ out,
-                                                                 long long o_tok, int o_head, int tail, int rot_dims,
+                                                                 long long o_tok, int o_head, int tail, int rot_dims, int halves,
                                                                  const float2* __restrict__ cs, int half, float mag, int n_tokens) {
     pdl_launch_dependents();
     pdl_wait();
@@ -127,25 +129,16 @@ __global__ void __launch_bounds__(HW_WARPS * 32) headwise_kernel(const float* __
         if (tt < nt && o < O) from_f32(out[(size_t)(t0 + tt) * o_tok + (size_t)h * o_head + o], s);
     }
     if (blockIdx.z != 0) return;
-    for (int e = threadIdx.x; e < nt * ((tail + 1) / 2); e += blockDim.x) {
-        const int tt = e / ((tail + 1) / 2), i = e % ((tail + 1) / 2), t = t0 + tt;
+    for (int e = threadIdx.x; e < nt * tail; e += blockDim.x) {
+        const int tt = e / tail, d = e % tail, t = t0 + tt;
         const float* xr = x + (size_t)t * x_tok + (size_t)h * x_head + I;
-        OutT* orow = out + (size_t)t * o_tok + (size_t)h * o_head + O;
-        float u = xr[2 * i], v = (2 * i + 1 < tail) ? xr[2 * i + 1] : 0.f;
-        if (2 * i + 1 < rot_dims) {
-            const float2 a = cs[(size_t)t * half + i];
-            const float co = a.x * mag, si = a.y * mag;
-            const float u2 = u * co - v * si, v2 = v * co + u * si;
-            u = u2; v = v2;
-        }
-        from_f32(orow[2 * i], u);
-        if (2 * i + 1 < tail) from_f32(orow[2 * i + 1], v);
+        from_f32(out[(size_t)t * o_tok + (size_t)h * o_head + O + d], latent_turned(xr, d, rot_dims, halves, cs + (size_t)t * half, mag));
     }
 }
 
 // out_is_f32: the outputs are 32-bit (queries in the latent's space); else the storage type (a product's input)
 extern "C" int idm_headwise(const float* x, long long x_tok, int x_head, int I, const void* W, int O, void* out,
-                            int out_is_f32, long long o_tok, int o_head, int tail, int rot_dims, const float* cs, int half,
+                            int out_is_f32, long long o_tok, int o_head, int tail, int rot_dims, int halves, const float* cs, int half,
                             float mag, int n_tokens, int n_heads, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
     IDM_REQUIRE(I > 0 && O >= 0 && n_heads > 0 && tail >= 0, "headwise: sizes I=%d O=%d heads=%d tail=%d", I, O, n_heads, tail);
@@ -158,11 +151,11 @@ extern "C" int idm_headwise(const float* x, long long x_tok, int x_head, int I, 
     if (out_is_f32) {
         if (smem > 48 * 1024) cudaFuncSetAttribute(headwise_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         idm_launch(headwise_kernel<float>, grid, dim3(HW_WARPS * 32), smem, stream, x, x_tok, x_head, I, (const T*)W, O, (float*)out,
-                   o_tok, o_head, tail, rot_dims, (const float2*)cs, half, mag, n_tokens);
+                   o_tok, o_head, tail, rot_dims, halves, (const float2*)cs, half, mag, n_tokens);
     } else {
         if (smem > 48 * 1024) cudaFuncSetAttribute(headwise_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         idm_launch(headwise_kernel<T>, grid, dim3(HW_WARPS * 32), smem, stream, x, x_tok, x_head, I, (const T*)W, O, (T*)out,
-                   o_tok, o_head, tail, rot_dims, (const float2*)cs, half, mag, n_tokens);
+                   o_tok, o_head, tail, rot_dims, halves, (const float2*)cs, half, mag, n_tokens);
     }
     IDM_LAUNCH_CHECK("headwise");
     return 0;
@@ -698,7 +691,7 @@ extern "C" int idm_latent_attention(const float* qa, const void* pool, const int
 // [Uk ; Uv]; rows: the step's packed [c | r] rows in the storage type.  One block per token.
 __global__ void __launch_bounds__(256) latent_expand_pack_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ up,
                                                                  const T* __restrict__ rows, int H, int dn, int dr, int dv, int R,
-                                                                 int rot_dims, const float2* __restrict__ cs, int half, float mag,
+                                                                 int rot_dims, int halves, const float2* __restrict__ cs, int half, float mag,
                                                                  int hd, T* __restrict__ q, T* __restrict__ k, T* __restrict__ v,
                                                                  const int* __restrict__ table, int table_stride,
                                                                  const int* __restrict__ token_seq, const int* __restrict__ positions,
@@ -722,12 +715,7 @@ __global__ void __launch_bounds__(256) latent_expand_pack_kernel(const float* __
         } else if (d < dn + dr) {
             const int j = d - dn;
             const float* qr = pq + h * (dn + dr) + dn;
-            qv = qr[j];
-            if ((j | 1) < rot_dims) {                       // the pair (j & ~1, j | 1) is turned
-                const float2 a = cs[(size_t)t * half + (j >> 1)];
-                const float co = a.x * mag, si = a.y * mag;
-                qv = (j & 1) ? qr[j] * co + qr[j - 1] * si : qr[j] * co - qr[j + 1] * si;
-            }
+            qv = latent_turned(qr, j, rot_dims, halves, cs + (size_t)t * half, mag);
             kk = r[j];
         }
         if (d < dv) from_f32(vv, pu[H * dn + h * dv + d]);
@@ -739,7 +727,7 @@ __global__ void __launch_bounds__(256) latent_expand_pack_kernel(const float* __
 }
 
 extern "C" int idm_latent_expand_pack(const float* proj, int ld, const float* up, const void* rows, int H, int dn, int dr,
-                                      int dv, int R, int rot_dims, const float* cs, int half, float mag, int hd, void* q,
+                                      int dv, int R, int rot_dims, int halves, const float* cs, int half, float mag, int hd, void* q,
                                       void* k, void* v, const int* table, int table_stride, const int* token_seq,
                                       const int* positions, const int* slots, int n_tokens, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
@@ -747,7 +735,7 @@ extern "C" int idm_latent_expand_pack(const float* proj, int ld, const float* up
                 dn, dr, dv, hd);
     IDM_REQUIRE(rot_dims >= 0 && rot_dims <= dr && rot_dims % 2 == 0 && (rot_dims == 0 || (cs != nullptr && half >= rot_dims / 2)),
                 "latent_expand_pack: %d turned dims of %d with a table of %d angles", rot_dims, dr, half);
-    idm_launch(latent_expand_pack_kernel, dim3(n_tokens), dim3(256), 0, stream, proj, ld, up, (const T*)rows, H, dn, dr, dv, R, rot_dims,
+    idm_launch(latent_expand_pack_kernel, dim3(n_tokens), dim3(256), 0, stream, proj, ld, up, (const T*)rows, H, dn, dr, dv, R, rot_dims, halves,
                (const float2*)cs, half, mag, hd, (T*)q, (T*)k, (T*)v, table, table_stride, token_seq, positions, slots);
     IDM_LAUNCH_CHECK("latent_expand_pack");
     return 0;

@@ -1,12 +1,13 @@
 // A learned router over feed-forward experts: from a token's logits over all experts (identity experts included) to
 // the experts it uses and their weights.
 //
-//   s      = softmax(z)                                   over all E experts, 32-bit
-//   c_e    = s_e + correction_e                           the score an expert is CHOSEN by
+//   s      = softmax(z) over all E experts, or sigmoid(z) element by element, 32-bit
+//   c_e    = s_e + correction_e                           the score an expert is CHOSEN by (sigmoids without a correction:
+//                                                         z itself, whose order is the same and which does not saturate)
 //   groups : E / count neighbours each; a group's score is its largest c; only experts of the `keep` best groups
 //            can be chosen (the others count as minus infinity)
 //   chosen : the `top` largest c among those, in descending order (ties: the lower index)
-//   weight : s_chosen / (sum of the chosen s + 1e-20) * scale
+//   weight : s_chosen / (sum of the chosen s + 1e-20) * scale, or (not renormalized) s_chosen * scale
 //
 // One warp per token; s and c wait in shared memory.  Nothing here depends on the other tokens of the step.
 #include "common.cuh"
@@ -26,7 +27,7 @@ __device__ __forceinline__ void warp_argmax(float& v, int& idx) {
 __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const float* __restrict__ z, int z_stride,
                                                               const float* __restrict__ correction, int* __restrict__ chosen,
                                                               float* __restrict__ weight, int n_tokens, int E, int top,
-                                                              int count, int keep, float scale) {
+                                                              int count, int keep, float scale, int sigmoid, int renorm) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ float sm[];
@@ -37,13 +38,21 @@ __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const float* __res
     float* c = s + E;                                            // [E] choice scores (minus infinity once taken or shut out)
     float* gs = c + E;                                           // [count] group scores
     const float* zr = z + (size_t)t * z_stride;
-    float m = -INFINITY;
-    for (int e = lane; e < E; e += 32) m = fmaxf(m, zr[e]);
-    m = warp_max(m);
-    float den = 0.f;
-    for (int e = lane; e < E; e += 32) { const float p = expf(zr[e] - m); s[e] = p; den += p; }
-    den = warp_sum(den);
-    for (int e = lane; e < E; e += 32) { s[e] = s[e] / den; c[e] = s[e] + (correction ? correction[e] : 0.f); }
+    if (sigmoid) {
+        for (int e = lane; e < E; e += 32) {
+            const float v = zr[e];
+            s[e] = 1.0f / (1.0f + expf(-v));
+            c[e] = correction ? s[e] + correction[e] : v;
+        }
+    } else {
+        float m = -INFINITY;
+        for (int e = lane; e < E; e += 32) m = fmaxf(m, zr[e]);
+        m = warp_max(m);
+        float den = 0.f;
+        for (int e = lane; e < E; e += 32) { const float p = expf(zr[e] - m); s[e] = p; den += p; }
+        den = warp_sum(den);
+        for (int e = lane; e < E; e += 32) { s[e] = s[e] / den; c[e] = s[e] + (correction ? correction[e] : 0.f); }
+    }
     __syncwarp();
     if (count > 1 && keep < count) {
         const int per = E / count;
@@ -81,12 +90,13 @@ __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const float* __res
         if (idx >= 0) total += s[idx];
         __syncwarp();
     }
-    const float f = scale / (total + 1e-20f);
+    const float f = renorm ? scale / (total + 1e-20f) : scale;
     for (int k = lane; k < top; k += 32) weight[(size_t)t * top + k] *= f;
 }
 
 extern "C" int idm_route(const float* z, int z_stride, const float* correction, int* chosen, float* weight, int n_tokens,
-                         int n_experts, int top, int groups, int keep, float scale, cudaStream_t stream) {
+                         int n_experts, int top, int groups, int keep, float scale, int sigmoid, int renorm,
+                         cudaStream_t stream) {
     if (n_tokens == 0) return 0;
     IDM_REQUIRE(n_experts > 0 && top > 0 && top <= n_experts && z_stride >= n_experts, "route: %d experts, %d per token, rows of %d",
                 n_experts, top, z_stride);
@@ -96,7 +106,7 @@ extern "C" int idm_route(const float* z, int z_stride, const float* correction, 
     IDM_REQUIRE(smem <= 160 * 1024, "route: %d experts do not fit shared memory", n_experts);
     if (smem > 48 * 1024) cudaFuncSetAttribute(route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     idm_launch(route_kernel, dim3((n_tokens + RT_WARPS - 1) / RT_WARPS), dim3(RT_WARPS * 32), smem, stream, z, z_stride, correction,
-               chosen, weight, n_tokens, n_experts, top, groups, keep, scale);
+               chosen, weight, n_tokens, n_experts, top, groups, keep, scale, sigmoid, renorm);
     IDM_LAUNCH_CHECK("route");
     return 0;
 }

@@ -60,7 +60,7 @@ SIGNATURES = {
     "idm_embed": (c_int, "pppiip"),
     "idm_embed_scaled": (c_int, "pppiifp"),
     "idm_post_pre_norm": (c_int, "pppfpfpiiip"),
-    "idm_gated_act": (c_int, "ppiiip"),
+    "idm_gated_act": (c_int, "ppiiipp"),
     "idm_token_gate": (c_int, "pppiipiiip"),
     "idm_short_conv": (c_int, "piiiippipqppppppip"),
     "idm_conv_qkv_cache": (c_int, "piiippqiiiiipppppipppppip"),
@@ -69,8 +69,8 @@ SIGNATURES = {
     "idm_ssd_scan": (c_int, "piiiipiiippppqpippiiiiippipip"),
     "idm_ssd_group_norm": (c_int, "piipffpiiip"),
     "idm_attention_sink": (c_int, "ppiifpppippipppppiiiiifip"),
-    "idm_attention_biased": (c_int, "ppiifpppiipppiipppppiiiiififip"),
-    "idm_head_finish": (c_int, "piiiipppppfipfiiiippppiipppip"),
+    "idm_attention_biased": (c_int, "ppiifpppiipppiipppppiiiiififiipp"),
+    "idm_head_finish": (c_int, "piiiipppppiiifipfiiiippppiipppip"),
     "idm_cols_cast": (c_int, "piiipiip"),
     "idm_delta_prep": (c_int, "piiipiipiiipppiiiip"),
     "idm_delta_scan": (c_int, "piiiipiippqpippiiiiiipp"),
@@ -78,6 +78,7 @@ SIGNATURES = {
     "idm_delta_out": (c_int, "pipfpiiifpiiiiip"),
     "idm_add_rmsnorm2": (c_int, "ppiqppfpppiip"),
     "idm_gemm_bf16_gated": (c_int, "pppiiiip"),
+    "idm_gemm_bf16_gated_rows": (c_int, "pppiiiipp"),
     "idm_add_rmsnorm": (c_int, "ppiqpfppiip"),
     "idm_rope_table": (c_int, "ppppiip"),
     "idm_qkv_finish": (c_int, "piqiiiippfpppppppiipppp"),
@@ -97,28 +98,30 @@ SIGNATURES = {
     "idm_attention_tc_scratch_floats": (c_longlong, "iiiiii"),
     "idm_attention_tc": (c_int, "ppppipippippppiiiifiiippiip"),
     "idm_attention_tc_sink": (c_int, "pppppipippippppiiiifiiippiip"),
-    "idm_attention_tc_biased": (c_int, "ppppifippipippippppiiiifiiippiip"),
+    "idm_attention_tc_biased": (c_int, "ppppifiipppipippippppiiiifiiippiip"),
     "idm_gate_scale": (c_int, "ppiifpiiiip"),
     "idm_attention_tc_status": (c_int, ""),
     "idm_attention_tc_set_few_rows": (c_int, "i"),
-    "idm_latent_kv_finish": (c_int, "piiiiipfpifppippppip"),
-    "idm_headwise": (c_int, "pqiipipiqiiipifiip"),
+    "idm_latent_kv_finish": (c_int, "piiiiiipfpifppippppip"),
+    "idm_headwise": (c_int, "pqiipipiqiiiipifiip"),
     "idm_latent_attention_max_rank": (c_int, ""),
     "idm_latent_attention_heads_per_block": (c_int, "iii"),
     "idm_latent_attention": (c_int, "pppippppppiiiifiip"),
-    "idm_latent_expand_pack": (c_int, "pippiiiiiipifippppipppip"),
-    "idm_experts_few": (c_int, "pppppqqqpppiiiiiifp"),
-    "idm_experts_major": (c_int, "pppppqqqppppiiiiiifp"),
+    "idm_latent_expand_pack": (c_int, "pippiiiiiiipifippppipppip"),
+    "idm_experts_few": (c_int, "pppppqqqpppiiiiiifip"),
+    "idm_experts_major": (c_int, "pppppqqqppppiiiiiifip"),
     "idm_rows_gather": (c_int, "pppiip"),
     "idm_experts_grouped": (c_int, "ppipqpqppiiip"),
-    "idm_experts_dense": (c_int, "ppppipqpqpppiiiiifp"),
-    "idm_experts_grouped_step": (c_int, "pppppipqpqppppiiiiifp"),
+    "idm_experts_dense": (c_int, "ppppipqpqpppiiiiifpp"),
+    "idm_experts_grouped_step": (c_int, "pppppipqpqppppiiiiifpp"),
     "idm_dense_ff": (c_int, "ppppppiiiip"),
     "idm_experts_combine": (c_int, "ppppiiifp"),
-    "idm_route": (c_int, "pipppiiiiifp"),
+    "idm_rows_weight": (c_int, "pppip"),
+    "idm_route": (c_int, "pipppiiiiifiip"),
     "idm_experts_identity": (c_int, "ppppiiiip"),
     "idm_post_layernorm": (c_int, "pppppfpiiip"),
     "idm_add_layernorm": (c_int, "ppiqppfppiip"),
+    "idm_sum_norm": (c_int, "ppiqfpfippiiip"),
     "idm_embed_bigram": (c_int, "ppppppppqppiiqqqp"),
     "idm_add_dyt": (c_int, "ppiqppfppiip"),
     "idm_act_cast": (c_int, "ppqip"),
@@ -268,13 +271,17 @@ class Kernels:
                                                hidden, self._stream()))
         return x
 
-    def gated_act(self, gu: torch.Tensor, act: int) -> torch.Tensor:
+    def gated_act(self, gu: torch.Tensor, act: int, row_w=None) -> torch.Tensor:
         """``act(gate) * up`` of a 32-bit gate/up product ``[N, 2 * inter]`` (gate columns, then up columns);
-        ``act``: 0 silu, 1 gelu (tanh form)."""
+        ``act``: 0 silu, 1 gelu (tanh form).  ``row_w [N]``: gate and up of a row are multiplied by it first."""
         self._need(gu, torch.float32, "gate-up")
         n, width = gu.shape
         y = torch.empty((n, width // 2), dtype=self.dtype, device=self.device)
-        self._check(self.lib.idm_gated_act(_p(gu), _p(y), n, width // 2, act, self._stream()))
+        if row_w is not None:
+            self._need(row_w, torch.float32, "row weights")
+            if row_w.numel() != n:
+                raise KernelError(f"{row_w.numel()} row weights for {n} rows")
+        self._check(self.lib.idm_gated_act(_p(gu), _p(y), n, width // 2, act, _p(row_w), self._stream()))
         return y
 
     def token_gate(self, s, tokens, table, col0: int, act: int) -> torch.Tensor:
@@ -400,27 +407,32 @@ class Kernels:
 
     def attention_biased(self, q, kv, ctx, scale: float, out, out_col: int, out_scale: float = 1.0, sink=None,
                          slopes=None, gate=None, gate_stride: int = 0, gate_per_head: bool = False, window=None,
-                         softcap: float = 0.0, keep_first: int = 0) -> None:
+                         softcap: float = 0.0, keep_first: int = 0, chunk=None, score_bias=None) -> None:
         """The general attention kernel with all of its options: ``sink`` [n_q] joins the denominator, ``slopes`` [n_q]
         times the distance to a key is taken off its score, ``window`` keys are seen (and, whatever the distance, the
         sequence's first ``keep_first``), scores are capped at ``softcap * tanh(score / softcap)``, the result is multiplied by
         ``sigmoid(gate)`` (one number per head at ``gate[t, head]`` or one per channel) and by ``out_scale`` and
-        stored at columns ``out_col ..`` of ``out``."""
+        stored at columns ``out_col ..`` of ``out``.  ``chunk``: only keys of the query's own chunk of so many positions
+        are seen; ``score_bias`` [n_q]: weights ``sigmoid(score + score_bias)`` instead of a softmax."""
         n, n_q, dk = q.shape
         self._check_kv(kv, kv.n_kv_heads, dk, kv.v_head_dim)
-        for name, t in (("sink", sink), ("slopes", slopes)):
+        for name, t in (("sink", sink), ("slopes", slopes), ("score_bias", score_bias)):
             if t is not None and (t.dtype != torch.float32 or t.numel() != n_q):
                 raise KernelError(f"attention: {name} must hold one 32-bit number per head")
         self._check(self.lib.idm_attention_biased(
             _p(q), _p(out), out.shape[1], out_col, float(out_scale), _p(kv.k), _p(kv.v), _p(kv.table), kv.table.shape[1],
             kv.ring, _p(sink), _p(slopes), _p(gate), gate_stride, 1 if gate_per_head else 0, _p(ctx.token_seq),
             _p(ctx.positions), _p(ctx.slots), _p(ctx.q_start), _p(ctx.cu_q), n, n_q, kv.n_kv_heads, dk, kv.v_head_dim,
-            float(scale), int(window) if window else 0, float(softcap or 0.0), int(keep_first or 0), self._stream()))
+            float(scale), int(window) if window else 0, float(softcap or 0.0), int(keep_first or 0), int(chunk or 0),
+            _p(score_bias), self._stream()))
 
     def head_finish(self, proj, col_q: int, col_k: int, col_v, n_q: int, n_kv: int, dk: int, dv: int, biases, gammas,
-                    eps: float, cs, mag: float, kv, ctx) -> torch.Tensor:
+                    eps: float, cs, mag: float, kv, ctx, norm_all: bool = False, v_norm: bool = False,
+                    pairs: bool = False) -> torch.Tensor:
         """Bias, norm per head and partial rotation of the q and k heads in columns of the 32-bit ``proj``; k and v to
-        the cache entry (``col_v`` None: the keys as projected are the values); returns q ``[N, n_q, dk]``."""
+        the cache entry (``col_v`` None: the keys as projected are the values); returns q ``[N, n_q, dk]``.
+        ``norm_all``: one norm over all heads of q, one over all of k (``gammas`` of those sizes); ``v_norm``: value heads
+        over their own root mean square; ``pairs``: the rotation turns neighbours instead of dims half the turned part apart."""
         self._need(proj, torch.float32, "projection")
         n, width = proj.shape
         self._check_kv(kv, n_kv, dk, dv)
@@ -429,10 +441,13 @@ class Kernels:
             raise KernelError(f"rotary table {tuple(cs.shape)} does not match {(n, half, 2)}")
         bq, bk, bv = biases
         gq, gk = gammas
+        for g_, heads in ((gq, n_q), (gk, n_kv)):
+            if g_ is not None and g_.numel() != (heads * dk if norm_all else dk):
+                raise KernelError(f"q/k norm weight has {g_.numel()} elements, expected {heads * dk if norm_all else dk}")
         q = torch.empty((n, n_q, dk), dtype=self.dtype, device=self.device)
         self._check(self.lib.idm_head_finish(
             _p(proj), width, col_q, col_k, -1 if col_v is None else col_v, _p(bq), _p(bk), _p(bv), _p(gq), _p(gk),
-            float(eps), half, _p(cs), float(mag), n_q, n_kv, dk, dv, _p(q), _p(kv.k), _p(kv.v), _p(kv.table),
+            1 if norm_all else 0, 1 if v_norm else 0, 1 if pairs else 0, float(eps), half, _p(cs), float(mag), n_q, n_kv, dk, dv, _p(q), _p(kv.k), _p(kv.v), _p(kv.table),
             kv.table.shape[1], kv.ring, _p(ctx.token_seq), _p(ctx.positions), _p(ctx.slots), n, self._stream()))
         return q
 
@@ -602,7 +617,7 @@ class Kernels:
         return self.attention_generic(q, kv, ctx, k_new, v_new, scale, window)
 
     def attention_tc(self, q, kv, ctx, scale: float, out=None, through_scratch=None, share=None, sink=None, slopes=None,
-                     window=None, softcap: float = 0.0, keep_first: int = 0) -> torch.Tensor:
+                     window=None, softcap: float = 0.0, keep_first: int = 0, chunk=None, score_bias=None) -> torch.Tensor:
         """Causal attention on the tensor cores: tiles of (128 / gp tokens) x (gp q-heads of one kv-head).
 
         Steps with few tokens per sequence (at most 32 rows a tile: single tokens above all) give every
@@ -614,20 +629,20 @@ class Kernels:
         if out is None:
             out = torch.empty((n, n_q * hd), dtype=self.dtype, device=self.device)
         (tile_seq, tile_start, n_tiles, rows_cap, max_runs, scratch, tile_pool, max_parts,
-         per) = self.attention_tc_plan(ctx, n_q, kv.n_kv_heads, hd, through_scratch, share)
+         per) = self.attention_tc_plan(ctx, n_q, kv.n_kv_heads, hd, through_scratch, share, chunk)
         rest = (_p(kv.k), _p(kv.v), kv.k.shape[0],
                 _p(kv.table), kv.table.shape[1], tile_seq, tile_start, n_tiles, _p(ctx.cu_q), _p(ctx.q_start),
                 _p(ctx.kv_len), _p(ctx.slots), n, n_q, kv.n_kv_heads,
                 hd, scale, self.attention_run_blocks, max_runs, rows_cap, scratch, tile_pool, max_parts, per,
                 self._stream())
-        if slopes is not None or window or softcap:
-            # a slope per q-head times the distance to a key off its score, and a window of keys a query sees (runs of
-            # key blocks before every window of a tile are not walked)
-            for name, t in (("sink", sink), ("slopes", slopes)):
+        if slopes is not None or window or softcap or chunk or score_bias is not None:
+            # a slope per q-head times the distance to a key off its score, a window of keys a query sees, or the query's
+            # chunk (runs of key blocks before every window or chunk of a tile are not walked), sigmoids for weights
+            for name, t in (("sink", sink), ("slopes", slopes), ("score_bias", score_bias)):
                 if t is not None and (t.dtype != torch.float32 or t.numel() != n_q):
                     raise KernelError(f"attention: {name} must hold one 32-bit number per head")
             self._check(self.lib.idm_attention_tc_biased(_p(q), _p(out), _p(sink), _p(slopes), int(window) if window else 0,
-                                                         float(softcap or 0.0), int(keep_first or 0), *rest))
+                                                         float(softcap or 0.0), int(keep_first or 0), int(chunk or 0), _p(score_bias), *rest))
         elif sink is None:
             self._check(self.lib.idm_attention_tc(_p(q), _p(out), *rest))
         else:
@@ -654,17 +669,19 @@ class Kernels:
         self._check(self.lib.idm_gate_scale(_p(o), (gate.data_ptr() if gate is not None else None), gate_stride, int(gate_group),
                                             float(scale), _p(out), out.shape[1], out_col, n, width, self._stream()))
 
-    def attention_tc_plan(self, ctx, n_q: int, n_kv: int, hd: int, through_scratch=None, share=None):
+    def attention_tc_plan(self, ctx, n_q: int, n_kv: int, hd: int, through_scratch=None, share=None, chunk=None):
         """What the attention launches of one step share, for one arrangement of heads: the list of tiles
         (on the device; made once a step), how the tiles' runs are spread over blocks, and the scratch.
         Returns (tile_seq, tile_start, n_tiles, rows_cap, max_runs, scratch, tile_pool, max_parts,
-        runs_per_part) as ``idm_attention_tc`` takes them (addresses as integers or None)."""
+        runs_per_part) as ``idm_attention_tc`` takes them (addresses as integers or None).  ``chunk``: queries see their own
+        chunk of positions only, so a tile's runs are those from its first row's chunk on."""
         gp = self.lib.idm_attention_tc_heads_per_tile(n_q, n_kv)
         tok = 128 // gp
         R = self.attention_run_blocks
         # (the spread of shared tiles over the pool depends on the number of head groups: layers with other head counts
         # have plans of their own)
-        memo_key = ("attention_tc_tiles", gp, n_q // gp)
+        chunk = int(chunk or 0)
+        memo_key = ("attention_tc_tiles", gp, n_q // gp, chunk)
         tiles = ctx.memo.get(memo_key)
         if tiles is None and ctx.single_token:
             # one tile per sequence: the same list for every step of that many sequences (kept, so that a
@@ -680,7 +697,9 @@ class Kernels:
             items = []
             for i, L in enumerate(ctx.host_q_lens):
                 for st in range(0, L, tok):
-                    items.append((ctx.host_starts[i] + min(st + tok - 1, L - 1), i, st))
+                    first, last = ctx.host_starts[i] + st, ctx.host_starts[i] + min(st + tok - 1, L - 1)
+                    left_out = (first - first % chunk) // (self.page * R) * (self.page * R) if chunk else 0
+                    items.append((last - left_out, i, st))             # (the tile's last position counted from its first run)
             items.sort(key=lambda t: -t[0])
             rows_cap = min(tok, max(ctx.host_q_lens)) * gp
             # Tiles with more key blocks than a fair share of the step's are shared by several blocks, each
@@ -708,6 +727,8 @@ class Kernels:
         # an upper bound of the key blocks any tile has (a captured step is replayed at growing lengths)
         longest = -(-ctx.max_kv_len // self.page)
         max_runs = -(-longest // R)
+        if chunk:                       # a tile's rows see at most a chunk and the tile's own tokens, from a run's border on
+            max_runs = min(max_runs, -(-(chunk + tok) // (self.page * R)) + 1)
         if through_scratch is None:
             # every run a block of its own where a tile has few rows (single tokens above all): the runs'
             # results are small then.  For whole tiles of a prompt the way through scratch was measured
@@ -982,9 +1003,10 @@ class Kernels:
         return int(self.lib.idm_latent_attention_max_rank())
 
     def latent_kv_finish(self, proj, col0: int, rank: int, rot_dim: int, rot_dims: int, w_norm, eps: float, cs, mag: float,
-                         kv, ctx, keep_rows: bool = False):
+                         kv, ctx, keep_rows: bool = False, halves: bool = False):
         """Columns ``[col0, col0 + rank + rot_dim)`` of the 32-bit ``proj``: the first ``rank`` normed (one root mean
-        square, times ``w_norm``), the rest turned by the step's table ``cs [N, half, 2]``; the row goes to the
+        square, times ``w_norm``), the rest turned by the step's table ``cs [N, half, 2]`` (neighbours, or with ``halves``
+        dims half the turned part apart); the row goes to the
         token's place in the cache entry and, with ``keep_rows``, is also returned packed ``[N, rank + rot_dim]``."""
         self._need(proj, torch.float32, "projection")
         n, ld = proj.shape
@@ -993,13 +1015,13 @@ class Kernels:
             raise KernelError(f"cache entry {tuple(kv.k.shape)} {kv.k.dtype} does not fit [pages, 1, {self.page}, {D}]")
         half = 0 if cs is None else cs.shape[1]
         rows = torch.empty((n, D), dtype=self.dtype, device=self.device) if keep_rows else None
-        self._check(self.lib.idm_latent_kv_finish(_p(proj), ld, col0, rank, rot_dim, rot_dims, _p(w_norm), eps, _p(cs), half,
+        self._check(self.lib.idm_latent_kv_finish(_p(proj), ld, col0, rank, rot_dim, rot_dims, 1 if halves else 0, _p(w_norm), eps, _p(cs), half,
                                                   float(mag), _p(kv.k), _p(kv.table), kv.table.shape[1], _p(ctx.token_seq),
                                                   _p(ctx.positions), _p(ctx.slots), _p(rows), n, self._stream()))
         return rows
 
     def headwise(self, x, x_col: int, n_heads: int, head_stride: int, w, tail: int = 0, rot_dims: int = 0, cs=None,
-                 mag: float = 1.0, out_f32: bool = False) -> torch.Tensor:
+                 mag: float = 1.0, out_f32: bool = False, halves: bool = False) -> torch.Tensor:
         """A matrix per head: ``out[t, h, :O] = x[t, x_col + h * head_stride : ... + I] . w[h]`` with ``w [H, I, O]``;
         ``tail`` more columns of ``x`` behind a head's ``I`` are copied behind its outputs, the first ``rot_dims`` of them
         turned.  ``x`` 32-bit ``[N, ld]``; returns ``[N, H, O + tail]`` (32-bit or the storage dtype)."""
@@ -1012,7 +1034,7 @@ class Kernels:
         out = torch.empty((n, H, O + tail), dtype=torch.float32 if out_f32 else self.dtype, device=self.device)
         half = 0 if cs is None else cs.shape[1]
         self._check(self.lib.idm_headwise(x.data_ptr() + 4 * x_col, ld, head_stride, I, _p(w), O, _p(out), 1 if out_f32 else 0,
-                                          H * (O + tail), O + tail, tail, rot_dims, _p(cs), half, float(mag), n, H,
+                                          H * (O + tail), O + tail, tail, rot_dims, 1 if halves else 0, _p(cs), half, float(mag), n, H,
                                           self._stream()))
         return out
 
@@ -1047,7 +1069,7 @@ class Kernels:
                                                   D, scale, run_keys, n_runs, self._stream()), 2 if n_runs > 1 else 1)
         return out
 
-    def latent_expand_pack(self, proj, up, rows, H, dn, dr, dv, R, rot_dims, cs, mag, hd, table, n_pages, ctx):
+    def latent_expand_pack(self, proj, up, rows, H, dn, dr, dv, R, rot_dims, cs, mag, hd, table, n_pages, ctx, halves: bool = False):
         """The operands of the per-head attention kernel for a step of whole prompts: ``q [N, H, hd]`` and pages of the
         step's own for k and v ``[n_pages, H, PAGE, hd]``, zero behind a head's own dims (see csrc/latent.cu)."""
         n = proj.shape[0]
@@ -1055,7 +1077,7 @@ class Kernels:
         k = torch.empty((n_pages, H, self.page, hd), dtype=self.dtype, device=self.device)
         v = torch.empty((n_pages, H, self.page, hd), dtype=self.dtype, device=self.device)
         half = 0 if cs is None else cs.shape[1]
-        self._check(self.lib.idm_latent_expand_pack(_p(proj), proj.shape[1], _p(up), _p(rows), H, dn, dr, dv, R, rot_dims, _p(cs),
+        self._check(self.lib.idm_latent_expand_pack(_p(proj), proj.shape[1], _p(up), _p(rows), H, dn, dr, dv, R, rot_dims, 1 if halves else 0, _p(cs),
                                                     half, float(mag), hd, _p(q), _p(k), _p(v), _p(table), table.shape[1],
                                                     _p(ctx.token_seq), _p(ctx.positions), _p(ctx.slots), n, self._stream()))
         return q, k, v
@@ -1065,11 +1087,11 @@ class Kernels:
     EXPERT_MAJOR_FROM = 64
 
     def experts_few(self, x, tokens, table, gate_up, row_stride: int, up_off: int, down, h, act: int, weight: float,
-                    pair_w=None) -> None:
+                    pair_w=None, weight_in: bool = False) -> None:
         """``h[t] += weight * sum_k down[e] (act(gate[e] x_t) * up[e] x_t)``, ``e = table[tokens[t], k]``: every (token, choice)
         streams its expert's matrices (steps of few tokens).  ``gate_up [E, rows, width]`` holds an expert's gate and up
         rows: gate row f starts ``f * row_stride`` elements into the expert's block and its up row ``up_off`` behind it.
-        ``down [E, width, ff]``."""
+        ``down [E, width, ff]``.  ``pair_w [N, top]`` weighs the pairs: their outputs, or with ``weight_in`` their inputs."""
         self._need(x, self.dtype, "experts input")
         self._need(h, torch.float32, "residual stream")
         self._need(gate_up, self.dtype, "experts' gate and up rows")
@@ -1088,10 +1110,10 @@ class Kernels:
             z = torch.zeros((n * top, width), dtype=torch.float32, device=self.device)
             self._check(self.lib.idm_experts_major(_p(x), _p(tokens), _p(table), _p(pair_w), _p(gate_up), gate_up.shape[1] * width, row_stride,
                                                    up_off, _p(down), _p(a), _p(z), _p(h), n, width, ff, top, E, act, float(weight),
-                                                   self._stream()), 3)
+                                                   1 if weight_in else 0, self._stream()), 3)
             return
         self._check(self.lib.idm_experts_few(_p(x), _p(tokens), _p(table), _p(pair_w), _p(gate_up), gate_up.shape[1] * width, row_stride, up_off, _p(down),
-                                             _p(a), _p(h), n, width, ff, top, E, act, float(weight), self._stream()), 2)
+                                             _p(a), _p(h), n, width, ff, top, E, act, float(weight), 1 if weight_in else 0, self._stream()), 2)
 
     def rows_gather(self, x, src) -> torch.Tensor:
         self._need(x, self.dtype, "rows")
@@ -1100,7 +1122,16 @@ class Kernels:
         self._check(self.lib.idm_rows_gather(_p(x), _p(src), _p(out), src.numel(), x.shape[1], self._stream()))
         return out
 
-    def experts_dense(self, x, tokens, table, gate_up, down, h, act: int, weight: float, pair_w=None) -> None:
+    def rows_weight(self, pair_w, place) -> torch.Tensor:
+        """The pairs' weights ``[N, top]`` in the order of the grouped rows: ``out[place[t, k]] = pair_w[t, k]``."""
+        self._need(pair_w, torch.float32, "pair weights")
+        self._need(place, torch.int32, "places")
+        out = torch.empty((place.numel(),), dtype=torch.float32, device=self.device)
+        self._check(self.lib.idm_rows_weight(_p(pair_w), _p(place), _p(out), place.numel(), self._stream()))
+        return out
+
+    def experts_dense(self, x, tokens, table, gate_up, down, h, act: int, weight: float, pair_w=None,
+                      weight_in: bool = False) -> None:
         """``h[t] += weight * sum_k ff_e(x_t)``, ``e = table[tokens[t], k]``, by running EVERY expert over all the step's
         tokens with the library's matrix products and letting each token pick its own (single-token steps of many
         sequences: every expert's matrices are streamed once, in shapes that do not change from step to step)."""
@@ -1110,11 +1141,13 @@ class Kernels:
         E, _, ff = down.shape
         y = torch.empty((n, ff), dtype=self.dtype, device=self.device)
         z = torch.empty((E, n, width), dtype=torch.float32, device=self.device)
+        w_in = torch.empty((E, n), dtype=torch.float32, device=self.device) if weight_in else None
         self._check(self.lib.idm_experts_dense(_p(x), _p(tokens), _p(table), _p(pair_w), E, _p(gate_up), gate_up.shape[1] * width, _p(down),
                                                width * ff, _p(y), _p(z), _p(h), n, width, ff, table.shape[1], act, float(weight),
-                                               self._stream()), 2 * E + 1)
+                                               _p(w_in), self._stream()), 2 * E + 1 + (1 if weight_in else 0))
 
-    def experts_grouped_step(self, x, src, place, counts, gate_up, down, h, act: int, weight: float, pair_w=None) -> None:
+    def experts_grouped_step(self, x, src, place, counts, gate_up, down, h, act: int, weight: float, pair_w=None,
+                             weight_in: bool = False) -> None:
         """A step's rows grouped by expert through every expert's gated feed-forward, from one call into the library:
         rows gathered in the order of their experts (``src [rows]``: grouped row -> token), the gated product (activation
         in its epilogue, ``gate_up`` in the layout of ``tile_gate_up``) and the down product of every expert that has
@@ -1128,10 +1161,12 @@ class Kernels:
         xg = torch.empty((n * top, width), dtype=self.dtype, device=self.device)
         y = torch.empty((n * top, ff), dtype=self.dtype, device=self.device)
         z = torch.empty((n * top, width), dtype=torch.float32, device=self.device)
+        row_w = torch.empty((n * top,), dtype=torch.float32, device=self.device) if weight_in else None
         with_rows = int((counts > 0).sum())
         self._check(self.lib.idm_experts_grouped_step(_p(x), _p(src), _p(place), _p(pair_w), counts.ctypes.data, E, _p(gate_up),
                                                       gate_up.shape[1] * width, _p(down), width * ff, _p(xg), _p(y), _p(z), _p(h),
-                                                      n, top, width, ff, act, float(weight), self._stream()), 2 * with_rows + 2)
+                                                      n, top, width, ff, act, float(weight), _p(row_w), self._stream()),
+                    2 * with_rows + 2 + (1 if weight_in else 0))
 
     def dense_ff(self, x, w_up, w_down, h, act: int) -> None:
         """``h += w_down . act(w_up . x)`` from one call: the up product, the activation, the down product with the sum
@@ -1152,11 +1187,12 @@ class Kernels:
         n, width = h.shape
         self._check(self.lib.idm_experts_combine(_p(z), _p(place), _p(pair_w), _p(h), n, width, place.shape[1], float(weight), self._stream()))
 
-    def route(self, z, correction, top: int, groups: int, keep: int, scale: float):
+    def route(self, z, correction, top: int, groups: int, keep: int, scale: float, sigmoid: bool = False, renorm: bool = True):
         """From 32-bit router logits ``z [N, E]`` to the experts each token uses: softmax over all E, choice by
         ``softmax + correction`` among the experts of the ``keep`` best of ``groups`` equal groups of neighbours, the
         ``top`` best in descending order; returns ``(chosen [N, top] int32, weight [N, top])`` with the weights the
-        chosen experts' softmax values over their sum, times ``scale``."""
+        chosen experts' softmax values over their sum, times ``scale``.  ``sigmoid``: element by element instead of the
+        softmax; ``renorm`` False: the chosen values times ``scale`` as they are."""
         self._need(z, torch.float32, "router logits")
         n, E = z.shape
         if correction is not None and (correction.dtype != torch.float32 or correction.numel() != E):
@@ -1164,7 +1200,7 @@ class Kernels:
         chosen = torch.empty((n, top), dtype=torch.int32, device=self.device)
         weight = torch.empty((n, top), dtype=torch.float32, device=self.device)
         self._check(self.lib.idm_route(_p(z), z.stride(0), _p(correction), _p(chosen), _p(weight), n, E, int(top), int(groups),
-                                       int(keep), float(scale), self._stream()))
+                                       int(keep), float(scale), 1 if sigmoid else 0, 1 if renorm else 0, self._stream()))
         return chosen, weight
 
     def experts_identity(self, x, chosen, weight, h, n_real: int) -> None:
@@ -1200,6 +1236,37 @@ class Kernels:
         x = torch.empty((n_out, hidden), dtype=self.dtype, device=self.device)
         self._check(self.lib.idm_add_layernorm(_p(h), dp, P, stride, _p(w), _p(b), float(eps), _p(x), _p(rows), n_out,
                                                hidden, self._stream()))
+        return x
+
+    def sum_norm(self, h, y, alpha: float, w, eps: float, groups: int = 1, cast: bool = True):
+        """``h <- N(alpha h + y)`` in place, ``N`` the RMS norm in ``groups`` equal parts times ``w``; ``y [P, N, hidden]`` 32-bit
+        partial sums.  Returns ``h`` in the storage dtype if ``cast``, else None."""
+        self._need(h, torch.float32, "residual stream")
+        self._need(w, torch.float32, "norm weight")
+        n, hidden = h.shape
+        if w.numel() != hidden or hidden % groups:
+            raise KernelError(f"sum_norm: rows of {hidden} in {groups} parts, weight of {w.numel()}")
+        yp, P, stride = self._delta_args(y, n, hidden)
+        x = torch.empty((n, hidden), dtype=self.dtype, device=self.device) if cast else None
+        self._check(self.lib.idm_sum_norm(_p(h), yp, P, stride, float(alpha), _p(w), float(eps), int(groups), _p(x), None, 1, n,
+                                          hidden, self._stream()))
+        return x
+
+    def grouped_rmsnorm(self, h, delta, w, eps: float, groups: int = 1, rows=None) -> torch.Tensor:
+        """The RMS norm in ``groups`` equal parts of ``h + delta`` (of the picked ``rows``) times ``w``, in the storage dtype;
+        the stream is left alone."""
+        self._need(h, torch.float32, "residual stream")
+        self._need(w, torch.float32, "norm weight")
+        n, hidden = h.shape
+        if w.numel() != hidden or hidden % groups:
+            raise KernelError(f"grouped_rmsnorm: rows of {hidden} in {groups} parts, weight of {w.numel()}")
+        dp, P, stride = self._delta_args(delta, n, hidden)
+        if rows is not None:
+            self._need(rows, torch.int32, "rows")
+        n_out = n if rows is None else rows.numel()
+        x = torch.empty((n_out, hidden), dtype=self.dtype, device=self.device)
+        self._check(self.lib.idm_sum_norm(_p(h), dp, P, stride, 1.0, _p(w), float(eps), int(groups), _p(x), _p(rows), 0, n_out,
+                                          hidden, self._stream()))
         return x
 
     def embed_bigram(self, ctx, table, bigram, last, buckets: int, mul_prev: int, mul_cur: int, cast: bool = False):

@@ -2,7 +2,7 @@
 
 from .base import (BLOCKS, EMBEDDINGS, FEED_FORWARDS, MIXERS, NORMS, POSITIONS, Block, CastStream, FeedForward, Mixer,
                    Norm, NormedDelta, Part, PositionEncoding, Runtime)
-from .norm import DyT, LayerNorm, RMSNorm
+from .norm import DyT, GroupedRMSNorm, LayerNorm, RMSNorm
 from .rotary import Rotary
 from .attention import GQAAttention
 from .mlp import DenseMLP, GatedMLP
@@ -15,6 +15,7 @@ from .latent_attention import LatentAttention
 from .experts import RoutedExperts, TableExperts
 from .embedding import BigramHashEmbedding
 from .postnorm_block import PostNormBlock
+from .sum_norm_block import SumNormBlock
 from .head_attention import HeadAttention
 from .delta_rule import GatedDeltaRule
 from .parallel_block import ParallelResidualBlock
@@ -24,4 +25,4 @@ __all__ = ["BLOCKS", "FEED_FORWARDS", "MIXERS", "NORMS", "POSITIONS", "Block", "
            "GatedMLP", "PreNormBlock", "SinkAttention", "SSDMixer", "ParallelMixer", "SandwichBlock", "TokenSide",
            "DyT", "DenseMLP", "LatentAttention", "TableExperts", "HeadAttention", "GatedDeltaRule",
            "ParallelResidualBlock", "EMBEDDINGS", "CastStream", "LayerNorm", "RoutedExperts", "BigramHashEmbedding",
-           "PostNormBlock"]
+           "PostNormBlock", "GroupedRMSNorm", "SumNormBlock"]

@@ -128,7 +128,11 @@ class RoutedExperts(FeedForward):
     the same kernels: a step's row numbers take the place of token ids and the step's choices the place of the table;
     every (token, choice) pair carries its weight.  Steps of many tokens, outside a captured graph, read the choices
     back and group the rows by expert for one matrix product per expert.  Returns the sum as a delta (a norm may sit
-    behind the feed-forward)."""
+    behind the feed-forward).
+
+    Options: ``s = sigmoid(z)`` instead of the softmax, no correction, weights left as they are (not over their sum), and
+    the weight on an expert's input, ``expert(w_k x_t)``: gate and up are linear, so w_k multiplies both of the pair's
+    pre-activations in 32-bit, in the epilogue of the product that makes them."""
 
     same_bits_across_steps = False      # whole prompts, portions and single tokens take different kernels
 
@@ -136,7 +140,9 @@ class RoutedExperts(FeedForward):
     def declare(cls, spec, prefix):
         s, nm = spec, spec.names
         total = s.n_experts + s.n_identity
-        d = [TensorDecl(prefix + s.router, (total, s.hidden)), TensorDecl(prefix + s.correction, (total,))]
+        d = [TensorDecl(prefix + s.router, (total, s.hidden))]
+        if s.correction is not None:
+            d.append(TensorDecl(prefix + s.correction, (total,)))
         for e in range(s.n_experts):
             p = prefix + s.expert.format(e)
             d += [TensorDecl(p + nm.gate, (s.intermediate, s.hidden)), TensorDecl(p + nm.up, (s.intermediate, s.hidden)),
@@ -154,6 +160,11 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"routed experts: {s.top} of {total} experts in {s.groups} groups of which {s.groups_keep} are kept")
         if s.top > s.groups_keep * (total // s.groups):
             raise ValueError(f"routed experts: {s.top} experts cannot come from {s.groups_keep} groups of {total // s.groups}")
+        if s.scores not in ("softmax", "sigmoid") or s.weight_on not in ("output", "input"):
+            raise ValueError(f"routed experts: scores={s.scores!r}, weight_on={s.weight_on!r} are not built")
+        if s.weight_on == "input" and s.n_identity:
+            raise ValueError("routed experts: a weight on the input and identity experts do not come together")
+        self.weight_in = s.weight_on == "input"
         self.spec, self.rt, self.act = spec, rt, ACTIVATIONS[s.activation]
         K = rt.kernels
 
@@ -172,7 +183,7 @@ class RoutedExperts(FeedForward):
                 self.row_stride, self.up_off = s.hidden, s.intermediate * s.hidden
             self.down = torch.stack(stack(nm.down)).contiguous()
         self.w_router = weights[prefix + s.router].to(rt.dtype).contiguous()
-        self.correction = weights[prefix + s.correction].to(torch.float32).contiguous()
+        self.correction = None if s.correction is None else weights[prefix + s.correction].to(torch.float32).contiguous()
         self.shared = None
         if s.shared is not None:
             self.shared = FEED_FORWARDS.get(s.shared.kind)(s.shared, weights, prefix, rt)
@@ -188,7 +199,8 @@ class RoutedExperts(FeedForward):
         """(chosen [N, top] int32, weight [N, top]) of the step's rows."""
         s, K = self.spec, self.rt.kernels
         z = K.gemm_store(x, self.w_router, pad=True)                        # 32-bit logits over all experts
-        return K.route(z, self.correction, s.top, s.groups, s.groups_keep, s.scale)
+        return K.route(z, self.correction, s.top, s.groups, s.groups_keep, s.scale, sigmoid=s.scores == "sigmoid",
+                       renorm=s.renormalize)
 
     def forward(self, x, ctx):
         s, K = self.spec, self.rt.kernels
@@ -205,10 +217,10 @@ class RoutedExperts(FeedForward):
             if in_eager_step and self.can_group and n * s.top >= GROUP_FROM:
                 self._grouped(x, chosen, weight, h)
             elif self.fused and n * s.top >= DENSE_FROM * s.n_experts:
-                K.experts_dense(x, rows, chosen, self.gate_up, self.down, h, self.act, 1.0, pair_w=weight)
+                K.experts_dense(x, rows, chosen, self.gate_up, self.down, h, self.act, 1.0, pair_w=weight, weight_in=self.weight_in)
             else:
                 K.experts_few(x, rows, chosen, self.gate_up, self.row_stride, self.up_off, self.down, h, self.act, 1.0,
-                              pair_w=weight)
+                              pair_w=weight, weight_in=self.weight_in)
         if s.n_identity:
             K.experts_identity(x, chosen, weight, h, s.n_experts)
         return h.unsqueeze(0)
@@ -227,8 +239,9 @@ class RoutedExperts(FeedForward):
         src, place_d = both[:n * top], both[n * top:].view(n, top)
         if self.fused:
             K.experts_grouped_step(x, src, place_d, np.ascontiguousarray(counts, dtype=np.int32), self.gate_up, self.down, h,
-                                   self.act, 1.0, pair_w=weight)
+                                   self.act, 1.0, pair_w=weight, weight_in=self.weight_in)
             return
+        row_w = K.rows_weight(weight, place_d) if self.weight_in else None
         xg = K.rows_gather(x, src)
         z = torch.empty((n * top, s.hidden), dtype=torch.float32, device=x.device)
         at = 0
@@ -236,7 +249,8 @@ class RoutedExperts(FeedForward):
             c = int(counts[e])
             if not c:
                 continue
-            y = K.gated_act(K.gemm_store(xg[at:at + c], self.gate_up[e], **self.pad), self.act)
+            y = K.gated_act(K.gemm_store(xg[at:at + c], self.gate_up[e], **self.pad), self.act,
+                            row_w=None if row_w is None else row_w[at:at + c])
             K.gemm_store(y, self.down[e], out=z[at:at + c], **self.pad)
             at += c
-        K.experts_combine(z, place_d, h, 1.0, pair_w=weight)
+        K.experts_combine(z, place_d, h, 1.0, pair_w=None if self.weight_in else weight)

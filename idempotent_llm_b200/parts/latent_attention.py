@@ -5,7 +5,8 @@ In this file's notation, for the mixer's input h of one sequence (positions t = 
     [qn_i | qr_i]_t = rows of Wq h_t                  ``plain_dim`` unrotated and ``rot_dim`` rotated dims per head
     [a_t | b_t]     = Wd h_t                          ``kv_rank`` and ``rot_dim`` numbers
     c_t             = a_t / sqrt(mean(a_t^2) + eps) * g
-    r_t             = turn(b_t, t),  qr <- turn(qr, t)        neighbours (2j, 2j+1) by angle t f_j, times a magnitude
+    r_t             = turn(b_t, t),  qr <- turn(qr, t)        pairs j by angle t f_j, times a magnitude: neighbours (2j, 2j+1),
+                                                              or dims (j, j + dims / 2)
     s_tj            = scale * (qn_i . Uk_i c_j + qr_i . r_j)   (j <= t)
     w_tj            = exp(s_tj) / (sum_j' exp(s_tj') [+ exp(sink_i)])
     out_t           = Wo [.. | Uv_i sum_j w_tj c_j | ..]
@@ -61,13 +62,14 @@ class LatentAttention(Mixer):
         if s.kv_rank > rt.kernels.latent_max_rank():
             raise ValueError(f"latent attention: a latent of {s.kv_rank} numbers is more than the kernels hold "
                              f"({rt.kernels.latent_max_rank()})")
-        self.rot_dims, self.position, self.magnitude = 0, None, 1.0
+        self.rot_dims, self.position, self.magnitude, self.halves = 0, None, 1.0, False
         if s.position is not None:
             variant = getattr(s.position, "variant", None)
-            if variant != "interleaved" or s.position.dim > s.rot_dim or s.position.dim % 2:
+            if variant not in ("interleaved", "half_partial") or s.position.dim > s.rot_dim or s.position.dim % 2:
                 raise ValueError(f"latent attention: position encoding variant {variant!r} over {s.position.dim} of "
                                  f"{s.rot_dim} dims is not built; the kernels turn neighbours (2j, 2j+1) of the rotated part "
-                                 f"('interleaved')")
+                                 f"('interleaved') or dims half the turned part apart ('half_partial')")
+            self.halves = variant == "half_partial"
             self.position = POSITIONS.get(s.position.kind)(s.position, weights, prefix, rt)
             self.rot_dims = s.position.dim
             self.magnitude = float(getattr(self.position, "magnitude", 1.0))
@@ -119,11 +121,11 @@ class LatentAttention(Mixer):
     def _whole_prompts(self, proj, cs, ctx, kv, residual):
         s, K, hd = self.spec, self.rt.kernels, self.tc_hd
         rows = K.latent_kv_finish(proj, self.q_cols, s.kv_rank, s.rot_dim, self.rot_dims, self.down_norm, s.eps, cs,
-                                  self.magnitude, kv, ctx, keep_rows=True)
+                                  self.magnitude, kv, ctx, keep_rows=True, halves=self.halves)
         up = K.gemm_store(rows, self.w_up)                                  # 32-bit [N, H * plain_dim + H * value_dim]
         table, n_pages = self._step_pages(ctx)
         q, k, v = K.latent_expand_pack(proj, up, rows, s.n_heads, s.plain_dim, s.rot_dim, s.value_dim, s.kv_rank,
-                                       self.rot_dims, cs, self.magnitude, hd, table, n_pages, ctx)
+                                       self.rot_dims, cs, self.magnitude, hd, table, n_pages, ctx, halves=self.halves)
         own = KVView(k=k, v=v, table=table, ring=0, n_kv_heads=s.n_heads, head_dim=hd, window=None)
         o = K.attention_tc(q, own, ctx, s.softmax_scale, sink=self.sink)    # [N, H * hd]
         if residual is not None:
@@ -141,10 +143,10 @@ class LatentAttention(Mixer):
         if self.tc_hd and not ctx.single_token and ctx.max_q_len >= self.WHOLE_FROM and not any(ctx.host_starts):
             return self._whole_prompts(proj, cs, ctx, kv, residual)
         K.latent_kv_finish(proj, self.q_cols, s.kv_rank, s.rot_dim, self.rot_dims, self.down_norm, s.eps, cs,
-                           self.magnitude, kv, ctx)
+                           self.magnitude, kv, ctx, halves=self.halves)
         # queries into the latent's space, their rotated part turned: [N, H, rank + rot_dim], 32-bit
         qa = K.headwise(proj, 0, s.n_heads, s.plain_dim + s.rot_dim, self.uk, tail=s.rot_dim, rot_dims=self.rot_dims,
-                        cs=cs, mag=self.magnitude, out_f32=True)
+                        cs=cs, mag=self.magnitude, out_f32=True, halves=self.halves)
         c = K.latent_attention(qa, kv, ctx, s.kv_rank, s.softmax_scale, sink=self.sink)     # 32-bit [N, H * rank]
         o = K.headwise(c, 0, s.n_heads, s.kv_rank, self.uv_t).view(x.shape[0], s.n_heads * s.value_dim)
         if residual is not None and getattr(K, "fused", False) and not self.pad:

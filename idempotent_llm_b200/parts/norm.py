@@ -1,5 +1,6 @@
 """Norms.  RMS norm: ``x / sqrt(mean(x^2) + eps) * weight``, all in 32-bit; and, at the end of the file, a norm
-without statistics (``DyT``: ``tanh(alpha x) * w + b``) and the layer norm with weight and bias.
+without statistics (``DyT``: ``tanh(alpha x) * w + b``), the layer norm with weight and bias, and the RMS norm in
+groups (``GroupedRMSNorm``: each of several equal parts of the row over its own root mean square).
 
 The reference's float form is ``x / sqrt(mean(x^2))`` (tests/test_ops.py:198-199,
 scripts/attribute_error.py:48-51) with the weight folded into the consumer
@@ -89,3 +90,28 @@ class LayerNorm(Norm):
             delta.add_into(h, self.rt.kernels)
             delta = None
         return self.rt.kernels.add_layernorm(h, delta, self.weight, self.bias, self.spec.eps, rows=rows)
+
+
+@NORMS.register("grouped_rmsnorm")
+class GroupedRMSNorm(Norm):
+    """Each of ``groups`` equal parts of the row over its own ``sqrt(mean(part^2) + eps)``, the whole times a weight, in
+    32-bit.  As the norm in front of a sublayer it adds a pending delta into the stream first."""
+
+    @classmethod
+    def declare(cls, spec, prefix):
+        return [TensorDecl(prefix + spec.weight, (spec.size,), init="one_plus_normal")]
+
+    def __init__(self, spec, weights, prefix, rt):
+        if spec.groups < 1 or spec.size % spec.groups:
+            raise ValueError(f"a row of {spec.size} cannot be cut into {spec.groups} equal parts")
+        self.spec, self.rt = spec, rt
+        self.weight = weights[prefix + spec.weight].to(torch.float32).contiguous()
+
+    def forward(self, h, delta, ctx, rows=None):
+        if isinstance(delta, (NormedDelta, CastStream)):
+            delta.add_into(h, self.rt.kernels)
+            delta = None
+        if delta is not None and rows is None:
+            h += delta.sum(dim=0)
+            delta = None
+        return self.rt.kernels.grouped_rmsnorm(h, delta, self.weight, self.spec.eps, self.spec.groups, rows=rows)

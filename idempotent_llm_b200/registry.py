@@ -81,6 +81,8 @@ def _register_builtin() -> None:
     register_architecture(FUGINEX, FuginexConfig)
     from .config.pununex import ARCHITECTURE as PUNUNEX, PununexConfig
     register_architecture(PUNUNEX, PununexConfig)
+    from .config.tosodra import ARCHITECTURE as TOSODRA, TosodraConfig
+    register_architecture(TOSODRA, TosodraConfig)
 
 
 _register_builtin()
