@@ -126,21 +126,23 @@ def kv_bytes_per_token(eng) -> int:
 
 def cache_bytes_read(lm, lens) -> float:
     """Bytes of keys and values a single-token step reads for sequences that hold ``lens`` tokens: every cache entry's
-    rows of the keys its layer sees (all, or the last `window`)."""
+    rows of the keys its layer sees (all, the last `window`, or those of the last token's `chunk`)."""
     import math
     eng, total = lm.engine, 0.0
-    windows = {}
+    windows, chunks = {}, {}
     for e in lm.model.spec.schedule:
         m = lm.model.spec.layers[e.layer].mixer
         for b in getattr(m, "branches", None) or [type("B", (), {"mixer": m})]:
             w = getattr(b.mixer, "window", None)
             if w:
                 windows[e.cache] = int(w)
+            if getattr(b.mixer, "chunk", None):
+                chunks[e.cache] = int(b.mixer.chunk)
     for g_ in eng.cache.groups:
         row = (math.prod(g_.need.key_row()) + math.prod(g_.need.value_row())) * g_.k.element_size()
         for entry in g_.entries:
-            w = windows.get(entry)
-            total += row * sum(min(n, w) if w else n for n in lens)
+            w, c = windows.get(entry), chunks.get(entry)
+            total += row * sum(min(n, w) if w else (n - 1) % c + 1 if c else n for n in lens)
     return total
 
 
@@ -181,7 +183,7 @@ def decode_point(lm, lens, steps: int, warmup: int, seed: int, repeats: int = 1,
     ms = statistics.median(times)
     sess.finish()
     mean_len = sum(l + warmup + repeats * steps / 2 for l in lens)
-    kv_read = (cache_bytes_read(lm, [l + warmup + repeats * steps / 2 for l in lens]) if getattr(cfg, "architecture", "") == "Fuginex"
+    kv_read = (cache_bytes_read(lm, [l + warmup + repeats * steps / 2 for l in lens]) if getattr(cfg, "architecture", "") in ("Fuginex", "Tosodra")
                else kv_bytes_per_token(eng) * mean_len)
     bytes_step = step_weight_bytes(lm, batch) + kv_read + 2 * batch * state_bytes_per_sequence(eng)
     toks = sess.tokens()
@@ -305,6 +307,32 @@ def pununex_prefill_flops(cfg, lens) -> float:
     return total + 2 * W * cfg.vocab * len(lens)
 
 
+def tosodra_prefill_flops(cfg, lens) -> float:
+    """The same count for a Tosodra configuration, per layer: the mixer's input and output projections (with the gate),
+    or the latent's joint projection and every head's keys and values from it; attention over the keys a query sees (those
+    of its chunk); the router, `top` experts and the shared expert."""
+    W, tokens, total = cfg.width, sum(lens), 0.0
+
+    def seen(t, chunk):
+        if not chunk or chunk >= t:
+            return t * (t + 1) // 2
+        return t // chunk * (chunk * (chunk + 1) // 2) + (t % chunk) * (t % chunk + 1) // 2
+    for L in cfg.layers:
+        linear = 0
+        if L.mlp is not None:
+            linear += W * L.mlp.experts + 3 * W * L.mlp.ff * L.mlp.top + 3 * W * (L.mlp.shared_ff or 0)
+        if L.type == "attention":
+            a = L.attention
+            linear += W * (a.heads * (a.dim + a.vdim) + a.kv_heads * (a.dim + a.vdim)) + a.heads * a.vdim * W
+            total += sum(a.heads * 2 * (a.dim + a.vdim) * seen(t, a.chunk) for t in lens)
+        else:
+            m = L.latent
+            linear += W * (m.heads * (m.dim + m.rot_dim) + m.kv_rank + m.rot_dim) + m.kv_rank * m.heads * (m.dim + m.vdim) + m.heads * m.vdim * W
+            total += sum(m.heads * 2 * (m.dim + m.rot_dim + m.vdim) * seen(t, None) for t in lens)
+        total += 2 * tokens * linear
+    return total + 2 * W * cfg.vocab * len(lens)
+
+
 def panodra_prefill_flops(cfg, lens) -> float:
     """The same count for a Panodra configuration, per layer run: the joint input projection, every head's keys and
     values from the latent, the output projection, causal attention per head over keys of dim + rot_dim and values of
@@ -348,6 +376,8 @@ def prefill_flops(cfg, lens) -> float:
         return fuginex_prefill_flops(cfg, lens)
     if getattr(cfg, "architecture", "") == "Pununex":
         return pununex_prefill_flops(cfg, lens)
+    if getattr(cfg, "architecture", "") == "Tosodra":
+        return tosodra_prefill_flops(cfg, lens)
     if hasattr(cfg, "layers") and not hasattr(cfg, "hidden_size"):
         return lunulix_prefill_flops(cfg, lens)
     H, L, V = cfg.hidden_size, cfg.num_hidden_layers, cfg.vocab_size
@@ -517,7 +547,7 @@ def decode_kernel_times(lm, lens, seed: int):
              "ssd_scan", "ssd_group_norm", "token_gate", "gated_act", "attention_lse_gate", "add_dyt", "latent_kv_finish",
              "headwise", "latent_attention", "experts_few", "act_cast", "concat_cast", "logit_cap", "add_rmsnorm2", "head_finish",
              "attention_biased", "cols_cast", "delta_prep", "delta_scan", "delta_out", "gate_scale", "embed_bigram", "post_layernorm",
-             "add_layernorm", "route", "experts_identity", "experts_dense", "experts_grouped_step", "conv_state_update"]
+             "add_layernorm", "route", "experts_identity", "sum_norm", "grouped_rmsnorm", "experts_dense", "experts_grouped_step", "conv_state_update"]
     names = [n for n in names if hasattr(K, n)]
     out, saved = {}, {n: getattr(K, n) for n in names}
     timing = [False]
@@ -552,13 +582,14 @@ def decode_kernel_times(lm, lens, seed: int):
     return {n: {"calls": c, "ms": round(ms, 4)} for n, (c, ms) in sorted(out.items(), key=lambda kv: -kv[1][1])}
 
 
-BESIDE = {"fuginex": "lunulix", "pununex": "fuginex"}      # a design's closest other one (default: qwen3)
+BESIDE = {"fuginex": "lunulix", "pununex": "fuginex", "tosodra": "pununex"}      # a design's closest other one (default: qwen3)
 
 
 def design_comparison(args) -> int:
-    """``--design lunulix`` / ``--design panodra`` / ``--design fuginex`` / ``--design pununex``: decode and prefill
+    """``--design lunulix`` / ``--design panodra`` / ``--design fuginex`` / ``--design pununex`` / ``--design tosodra``: decode and prefill
     throughput of that design beside the closest other one (Qwen3; for Fuginex, Lunulix: an attention and a recurrence
-    side by side; for Pununex, Fuginex: a windowed attention beside a delta rule) at equal width,
+    side by side; for Pununex, Fuginex: a windowed attention beside a delta rule; for Tosodra, Pununex: norms behind the
+    sublayers, a bounded attention and routed experts) at equal width,
     depth (layer runs), heads, feed-forward size and vocabulary (random weights), with where a step's time goes kernel by
     kernel."""
     import torch
@@ -619,7 +650,7 @@ def main() -> int:
     ap.add_argument("--repeats", type=int, default=5, help="timed regions of --steps steps; the median counts")
     ap.add_argument("--skip-points", action="store_true", help="leave out decode at batch 1 and 64 and the 32-bit check")
     ap.add_argument("--skip-sizes", action="store_true", help="leave out the points at 8B and 32B layer sizes")
-    ap.add_argument("--design", default="", choices=["", "lunulix", "panodra", "fuginex", "pununex"],
+    ap.add_argument("--design", default="", choices=["", "lunulix", "panodra", "fuginex", "pununex", "tosodra"],
                     help="instead of the default workload: this design beside its closest other one at equal layer sizes")
     ap.add_argument("--design-sizes", default="0.6b,8b", help="layer sizes of --design (presets <design>-<size>)")
     args = ap.parse_args()

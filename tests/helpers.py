@@ -533,3 +533,102 @@ def make_pununex_dir(cfg: dict, out_dir: str, seed: int = 1, dtype=torch.bfloat1
         del f
         write_safetensors(path, tensors)
     return out_dir
+
+
+# ------------------------------------------------------------------------------------- Tosodra
+def tosodra_attention(heads=4, kv_heads=2, dim=24, vdim=16, scale=0.3, chunk=20, rot_dims=8, rot_base=5000.0, mlp="moe"):
+    """One ``attention`` layer of a Tosodra config.json; ``mlp``: None, "moe", or a dict as config.json has it."""
+    m = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=scale, rot=dict(base=rot_base, dims=rot_dims))
+    if chunk:
+        m["mask"] = dict(size=chunk)
+    return dict(type="attention", mixer=m, mlp=tosodra_moe() if mlp == "moe" else mlp)
+
+
+def tosodra_latent(heads=3, dim=16, rot_dim=8, vdim=24, kv_rank=40, scale=0.25, rot_base=3e4, mlp="moe"):
+    """One ``latent_attention`` layer; its rotated part is turned whole."""
+    m = dict(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=kv_rank, scale=scale, rot=dict(base=rot_base, dims=rot_dim))
+    return dict(type="latent_attention", mixer=m, mlp=tosodra_moe() if mlp == "moe" else mlp)
+
+
+def tosodra_moe(experts=6, top=2, ff=24, shared=40):
+    d = dict(kind="moe", expert=dict(ff=ff), router=dict(experts=experts, top=top))
+    if shared:
+        d["shared"] = dict(ff=shared)
+    return d
+
+
+def tosodra_config(layers, vocab=97, width=32, eps=1e-5, groups=4, alpha=1.7, emb_scale=3.0):
+    import copy
+    return dict(architecture="Tosodra", vocab=vocab, width=width, norm=dict(eps=eps, groups=groups), postln_alpha=alpha,
+                embedding=dict(scale=emb_scale), layers=[copy.deepcopy(L) for L in layers])
+
+
+# Small Tosodra models that differ from one another in every size and option.
+TOSODRA = {
+    # both kinds of layer in both orders, grouped heads, chunks shorter than a page, a layer without feed-forward
+    "A": lambda: tosodra_config([tosodra_attention(), tosodra_latent(), tosodra_attention(chunk=33, rot_dims=24, mlp=None),
+                                 tosodra_attention(heads=6, kv_heads=1, dim=10, vdim=14, rot_dims=2, mlp=tosodra_moe(experts=9, top=4, ff=40, shared=16))]),
+    # values of 1: one head everywhere, one expert of one, one part in the norm, constants of 1, chunks of one key
+    "B": lambda: tosodra_config([tosodra_latent(heads=1, dim=8, rot_dim=2, vdim=8, kv_rank=8, scale=1.0,
+                                                mlp=tosodra_moe(experts=1, top=1, ff=8, shared=8)),
+                                 tosodra_attention(heads=1, kv_heads=1, dim=8, vdim=8, scale=1.0, chunk=1, rot_dims=2,
+                                                   mlp=tosodra_moe(experts=2, top=1, ff=16, shared=8))],
+                                vocab=50, width=24, groups=1, alpha=1.0, emb_scale=1.0),
+    # widths that are no multiple of 8 (bfloat16 rows off the 16-byte borders), norm parts of ten elements, every expert
+    # chosen, chunks of one page and one key, a latent off the borders
+    "C": lambda: tosodra_config([tosodra_attention(heads=3, kv_heads=3, dim=12, vdim=6, scale=0.2, chunk=65, rot_dims=12,
+                                                   mlp=tosodra_moe(experts=3, top=3, ff=12, shared=20)),
+                                 tosodra_latent(heads=5, dim=6, rot_dim=10, vdim=10, kv_rank=22, scale=0.3,
+                                                mlp=tosodra_moe(experts=5, top=2, ff=20, shared=12))],
+                                vocab=33, width=20, eps=1e-6, groups=2, alpha=3.0, emb_scale=11.0),
+    # head sizes the tensor-core attention has, chunks of one page and of more than a run of key blocks, many experts
+    "T": lambda: tosodra_config([tosodra_attention(heads=4, kv_heads=1, dim=64, vdim=64, scale=0.12, chunk=64, rot_dims=16,
+                                                   mlp=tosodra_moe(experts=12, top=3, ff=32, shared=64)),
+                                 tosodra_attention(heads=2, kv_heads=2, dim=128, vdim=128, scale=0.09, chunk=700, rot_dims=128, mlp=None),
+                                 tosodra_latent(heads=4, dim=48, rot_dim=16, vdim=64, kv_rank=64, scale=0.125,
+                                                mlp=tosodra_moe(experts=20, top=1, ff=64, shared=32)),
+                                 tosodra_attention(heads=8, kv_heads=4, dim=64, vdim=64, scale=0.12, chunk=150, rot_dims=64)],
+                                vocab=211, width=96, groups=3, alpha=2.2, emb_scale=7.0),
+}
+
+
+def tosodra_random_config(seed: int) -> dict:
+    """A Tosodra configuration drawn from sizes a model of the design may have: one to four layers of both kinds in any
+    order, grouped and ungrouped heads, chunks below, at and above a page, part or all of a head turned, norms in any
+    number of parts, experts from one to many."""
+    import random
+    r = random.Random(seed)
+
+    def mlp():
+        if r.random() < 0.2:
+            return None
+        e = r.choice([1, 2, 4, 7, 16, 24])
+        return tosodra_moe(experts=e, top=r.randint(1, min(4, e)), ff=r.choice([16, 40, 64]), shared=r.choice([16, 32, 72]))
+
+    def layer():
+        if r.random() < 0.4:
+            return tosodra_latent(heads=r.choice([1, 2, 4, 6]), dim=r.choice([16, 32, 64]), rot_dim=r.choice([8, 16, 32]),
+                                  vdim=r.choice([16, 32, 64, 80]), kv_rank=r.choice([32, 64, 96, 160]), scale=r.choice([0.1, 0.2, 0.15]),
+                                  rot_base=r.choice([1e4, 1e6]), mlp=mlp())
+        kv = r.choice([1, 2, 4]); dim = r.choice([32, 48, 64, 128])
+        return tosodra_attention(heads=kv * r.choice([1, 2, 3, 4]), kv_heads=kv, dim=dim, vdim=r.choice([dim, dim, 16, 40]),
+                                 scale=r.choice([dim ** -0.5, 0.1, 0.2]), chunk=r.choice([7, 48, 64, 70, 129, 200, 1000]),
+                                 rot_dims=r.choice([2, 16, dim // 2, dim]), rot_base=r.choice([1e4, 4e5, 1e6]), mlp=mlp())
+    width = r.choice([64, 96, 128, 240])
+    return tosodra_config([layer() for _ in range(r.choice([1, 2, 3, 4]))], vocab=r.choice([128, 500, 1000]), width=width,
+                          eps=r.choice([1e-5, 1e-6]), groups=r.choice([1, 2, 4, 8]), alpha=r.choice([1.0, 1.6, 2.9]),
+                          emb_scale=r.choice([1.0, 6.0, 20.0]))
+
+
+def make_tosodra_dir(cfg: dict, out_dir: str, seed: int = 1, dtype=torch.bfloat16, std: float = 0.15, edit=None) -> str:
+    """A Tosodra model folder with seeded random weights; ``edit(name, tensor) -> tensor`` may change them."""
+    from idempotent_llm_b200.config import TosodraConfig
+    from idempotent_llm_b200.weights import write_random_model, write_safetensors, SafetensorsFile
+    write_random_model(TosodraConfig.from_dict(cfg), out_dir, seed=seed, dtype=dtype, std=std)
+    if edit is not None:
+        path = os.path.join(out_dir, "model.safetensors")
+        f = SafetensorsFile(path)
+        tensors = [(n, edit(n, f.get(n).clone())) for n in f.names()]
+        del f
+        write_safetensors(path, tensors)
+    return out_dir
