@@ -449,20 +449,25 @@ extern "C" int idm_swiglu(const float* gu, int n_partials, long long partial_str
 // ------------------------------------------------------------ scaled embedding
 // h[t, :] = table[tokens[t], :] * scale, the product rounded once in 32-bit
 __global__ void embed_scaled_kernel(const int* __restrict__ tokens, const T* __restrict__ table,
-                                    float* __restrict__ h, int hidden, float scale) {
+                                    float* __restrict__ h, T* __restrict__ x, int hidden, float scale) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
     const T* row = table + (size_t)tokens[t] * hidden;
     float* out = h + (size_t)t * hidden;
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) out[i] = to_f32(row[i]) * scale;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+        const float v = to_f32(row[i]) * scale;
+        out[i] = v;
+        if (x) from_f32(x[(size_t)t * hidden + i], v);
+    }
 }
 
-extern "C" int idm_embed_scaled(const int* tokens, const void* table, float* h, int n_tokens, int hidden,
+// x (or null): the same rows in the storage type, for a first sublayer that reads the stream itself
+extern "C" int idm_embed_scaled(const int* tokens, const void* table, float* h, void* x, int n_tokens, int hidden,
                                 float scale, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
     IDM_REQUIRE(n_tokens > 0 && hidden > 0, "embed: bad sizes n_tokens=%d hidden=%d", n_tokens, hidden);
-    idm_launch(embed_scaled_kernel, dim3(n_tokens), dim3(256), 0, stream, tokens, (const T*)table, h, hidden, scale);
+    idm_launch(embed_scaled_kernel, dim3(n_tokens), dim3(256), 0, stream, tokens, (const T*)table, h, (T*)x, hidden, scale);
     IDM_LAUNCH_CHECK("embed_scaled");
     return 0;
 }

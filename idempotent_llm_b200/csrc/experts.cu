@@ -19,14 +19,24 @@ __device__ __forceinline__ float pair_act(float g, float u, float pw, int weight
     return weight_in ? gated_act(g * pw, u * pw, act) : gated_act(g, u, act) * pw;
 }
 
+// s + sum over a 16-byte piece of a row of its elements times x's, in ascending order; x (in shared memory, on a 16-byte
+// border) is read four numbers at a time: element by element, a warp's lanes would meet in the same banks
+__device__ __forceinline__ float piece_dot(const Vec16<T>& w, const float* __restrict__ x, float s) {
+#pragma unroll
+    for (int e = 0; e < Vec16<T>::N; e += 4) {
+        const float4 v = *reinterpret_cast<const float4*>(x + e);
+        s = fmaf(v.x, w.get(e), s); s = fmaf(v.y, w.get(e + 1), s); s = fmaf(v.z, w.get(e + 2), s); s = fmaf(v.w, w.get(e + 3), s);
+    }
+    return s;
+}
+
 __device__ __forceinline__ float row_dot(const T* __restrict__ w, const float* __restrict__ xs, int K, int lane, bool vec) {
     float s = 0.f;
     if (vec) {
         constexpr int VN = Vec16<T>::N;
         for (int d = lane * VN; d < K; d += 32 * VN) {
             Vec16<T> wv; wv.load(w + d);
-#pragma unroll
-            for (int e = 0; e < VN; ++e) s = fmaf(xs[d + e], wv.get(e), s);
+            s = piece_dot(wv, xs + d, s);
         }
     } else {
         for (int d = lane; d < K; d += 32) s = fmaf(xs[d], to_f32(w[d]), s);
@@ -47,26 +57,21 @@ __device__ __forceinline__ void row_dot2(const T* __restrict__ w0, const T* __re
 #pragma unroll
             for (int c = 0; c < 4; ++c) { a[c].load(w0 + d + c * 32 * VN); b[c].load(w1 + d + c * 32 * VN); }
 #pragma unroll
-            for (int c = 0; c < 4; ++c)
-#pragma unroll
-                for (int e = 0; e < VN; ++e) {
-                    s0 = fmaf(x0[d + c * 32 * VN + e], a[c].get(e), s0);
-                    s1 = fmaf(x1[d + c * 32 * VN + e], b[c].get(e), s1);
-                }
+            for (int c = 0; c < 4; ++c) {
+                s0 = piece_dot(a[c], x0 + d + c * 32 * VN, s0);
+                s1 = piece_dot(b[c], x1 + d + c * 32 * VN, s1);
+            }
         }
         for (; d + 32 * VN < K; d += 64 * VN) {
             Vec16<T> a0, a1, b0, b1;
             a0.load(w0 + d); b0.load(w1 + d); a1.load(w0 + d + 32 * VN); b1.load(w1 + d + 32 * VN);
-#pragma unroll
-            for (int e = 0; e < VN; ++e) { s0 = fmaf(x0[d + e], a0.get(e), s0); s1 = fmaf(x1[d + e], b0.get(e), s1); }
-#pragma unroll
-            for (int e = 0; e < VN; ++e) { s0 = fmaf(x0[d + 32 * VN + e], a1.get(e), s0); s1 = fmaf(x1[d + 32 * VN + e], b1.get(e), s1); }
+            s0 = piece_dot(a0, x0 + d, s0); s1 = piece_dot(b0, x1 + d, s1);
+            s0 = piece_dot(a1, x0 + d + 32 * VN, s0); s1 = piece_dot(b1, x1 + d + 32 * VN, s1);
         }
         for (; d < K; d += 32 * VN) {
             Vec16<T> a0, b0;
             a0.load(w0 + d); b0.load(w1 + d);
-#pragma unroll
-            for (int e = 0; e < VN; ++e) { s0 = fmaf(x0[d + e], a0.get(e), s0); s1 = fmaf(x1[d + e], b0.get(e), s1); }
+            s0 = piece_dot(a0, x0 + d, s0); s1 = piece_dot(b0, x1 + d, s1);
         }
     } else {
         for (int d = lane; d < K; d += 32) { s0 = fmaf(x0[d], to_f32(w0[d]), s0); s1 = fmaf(x1[d], to_f32(w1[d]), s1); }
@@ -86,7 +91,7 @@ __global__ void __launch_bounds__(256) experts_gate_up_kernel(const T* __restric
                                                               int act, int weight_in) {
     pdl_launch_dependents();
     pdl_wait();
-    extern __shared__ float xs[];
+    extern __shared__ __align__(16) float xs[];
     const int tk = blockIdx.x;
     const int t = tk / top;
     const int e = table[(size_t)tokens[t] * top + tk % top];       // the token's id names its experts
@@ -111,7 +116,7 @@ __global__ void __launch_bounds__(256) experts_down_kernel(const float* __restri
                                                            int ff, int top, int n_experts, float weight) {
     pdl_launch_dependents();
     pdl_wait();
-    extern __shared__ float as[];                             // [top][ff]
+    extern __shared__ __align__(16) float as[];                             // [top][ff]
     const int t = blockIdx.x;
     for (int d = threadIdx.x; d < top * ff; d += blockDim.x) as[d] = a[(size_t)t * top * ff + d];
     __syncthreads();

@@ -76,6 +76,7 @@ class CausalLM:
         self.final_norm = NORMS.get(spec.final_norm.kind)(spec.final_norm, weights,
                                                           spec.final_norm_prefix, rt)
         self.mix_in = weights[spec.mix_in_name].to(rt.dtype).contiguous() if spec.mix_in_name else None
+        self.stream_first = bool(getattr(self.blocks[spec.schedule[0].layer], "reads_stream", False)) if spec.schedule else False
         self._programs = {}
         self.graph_safe = all(getattr(part, "graph_safe", True) for b in self.blocks
                               for part in vars(b).values())
@@ -135,6 +136,9 @@ class CausalLM:
         pending = None
         if self.embedding is not None:
             h, pending = self.embedding.forward(self.embed, ctx, cache.state_of(EMBEDDING_CACHE_ID))
+        elif self.stream_first and self.mix_in is None:     # the first sublayer reads the stream itself: cast in the same pass
+            h, x = K.embed_scaled(ctx.tokens, self.embed, scale, cast=True)
+            pending = CastStream(x)
         else:
             h = K.embed(ctx.tokens, self.embed) if scale == 1.0 else K.embed_scaled(ctx.tokens, self.embed, scale)
         pad = {"pad": True} if self.spec.hidden % 8 else {}

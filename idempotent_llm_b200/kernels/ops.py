@@ -58,7 +58,7 @@ SIGNATURES = {
     "idm_page_tokens": (c_int, ""),
     "idm_set_pdl": (None, "i"),
     "idm_embed": (c_int, "pppiip"),
-    "idm_embed_scaled": (c_int, "pppiifp"),
+    "idm_embed_scaled": (c_int, "ppppiifp"),
     "idm_post_pre_norm": (c_int, "pppfpfpiiip"),
     "idm_gated_act": (c_int, "ppiiipp"),
     "idm_token_gate": (c_int, "pppiipiiip"),
@@ -248,14 +248,15 @@ class Kernels:
                                        n, hidden, self._stream()))
         return h
 
-    def embed_scaled(self, tokens: torch.Tensor, table: torch.Tensor, scale: float) -> torch.Tensor:
-        """``table[tokens] * scale`` as the 32-bit stream."""
+    def embed_scaled(self, tokens: torch.Tensor, table: torch.Tensor, scale: float, cast: bool = False):
+        """``table[tokens] * scale`` as the 32-bit stream; with ``cast`` also in the storage dtype: ``(h, x)``."""
         self._need(tokens, torch.int32, "embed tokens")
         self._need(table, self.dtype, "embed table")
         n, hidden = tokens.numel(), table.shape[1]
         h = torch.empty((n, hidden), dtype=torch.float32, device=self.device)
-        self._check(self.lib.idm_embed_scaled(_p(tokens), _p(table), _p(h), n, hidden, float(scale), self._stream()))
-        return h
+        x = torch.empty((n, hidden), dtype=self.dtype, device=self.device) if cast else None
+        self._check(self.lib.idm_embed_scaled(_p(tokens), _p(table), _p(h), _p(x), n, hidden, float(scale), self._stream()))
+        return (h, x) if cast else h
 
     def post_pre_norm(self, h, y, w_post, eps: float, w_pre=None, eps_pre: float = 0.0, cast: bool = False):
         """``h += rmsnorm(y) * w_post`` in place; returns what the next sublayer reads: ``rmsnorm(h) * w_pre`` if
@@ -681,7 +682,7 @@ class Kernels:
         # (the spread of shared tiles over the pool depends on the number of head groups: layers with other head counts
         # have plans of their own)
         chunk = int(chunk or 0)
-        memo_key = ("attention_tc_tiles", gp, n_q // gp, chunk)
+        memo_key = ("attention_tc_tiles", gp, n_q // gp) + ((chunk,) if chunk else ())
         tiles = ctx.memo.get(memo_key)
         if tiles is None and ctx.single_token:
             # one tile per sequence: the same list for every step of that many sequences (kept, so that a
@@ -1084,7 +1085,7 @@ class Kernels:
 
     # ---- experts chosen per token -------------------------------------------------------------------
     # from this many (token, choice) pairs on, a step of few tokens walks its experts one by one
-    EXPERT_MAJOR_FROM = 64
+    EXPERT_MAJOR_FROM = 256
 
     def experts_few(self, x, tokens, table, gate_up, row_stride: int, up_off: int, down, h, act: int, weight: float,
                     pair_w=None, weight_in: bool = False) -> None:

@@ -23,9 +23,18 @@ from .mlp import ACTIVATIONS
 
 # steps with at least this many (token, choice) pairs group their rows by expert (where the host has the tokens)
 GROUP_FROM = 256
-# steps that cannot group (their token ids are on the device only) with at least this many (token, choice) pairs per
-# expert run every expert over all tokens with the library's matrix products
-DENSE_FROM = 4
+# steps that cannot group (their token ids, or choices, are on the device only) with at least this many (token, choice)
+# pairs per expert run every expert over all tokens with the library's matrix products.  A pair that streams its expert pays
+# for the bytes, an expert's two products for their launches: experts of 5 MB break even at about 13 pairs each (16 of
+# them, 128 pairs: 99 us against 161 us; 256 pairs: 185 us against 169 us), experts of 75 MB at about 3.
+DENSE_FROM = 12
+LARGE_EXPERT, DENSE_FROM_LARGE = 16 << 20, 3
+
+
+def dense_from(spec, dtype) -> float:
+    """(token, choice) pairs from which a step that cannot group runs every expert over all its tokens."""
+    size = 3 * spec.hidden * spec.intermediate * torch.empty((), dtype=dtype).element_size()
+    return (DENSE_FROM_LARGE if size >= LARGE_EXPERT else DENSE_FROM) * spec.n_experts
 
 
 @FEED_FORWARDS.register("table_experts")
@@ -67,6 +76,7 @@ class TableExperts(FeedForward):
         self.down = torch.stack(stack(nm.down)).contiguous()
         self.table = weights[prefix + s.table].to(torch.int32).contiguous()
         self.table_host = self.table.cpu().numpy()
+        self.dense_from = dense_from(s, rt.dtype)
         bad = (self.table_host < 0) | (self.table_host >= s.n_experts)
         if bad.any():
             raise ValueError(f"{prefix + s.table}: entries outside the {s.n_experts} experts")
@@ -82,7 +92,7 @@ class TableExperts(FeedForward):
             if ids is None:
                 ids = ctx.memo["host_token_array"] = np.concatenate([np.asarray(t, dtype=np.int64) for t in toks])
             self._grouped(x, ids, h)
-        elif self.fused and n * s.top >= DENSE_FROM * s.n_experts:
+        elif self.fused and n * s.top >= self.dense_from:
             K.experts_dense(x, ctx.tokens, self.table, self.gate_up, self.down, h, self.act, 1.0 / s.top)
         else:
             K.experts_few(x, ctx.tokens, self.table, self.gate_up, self.row_stride, self.up_off, self.down, h, self.act, 1.0 / s.top)
@@ -187,6 +197,7 @@ class RoutedExperts(FeedForward):
         self.shared = None
         if s.shared is not None:
             self.shared = FEED_FORWARDS.get(s.shared.kind)(s.shared, weights, prefix, rt)
+        self.dense_from = dense_from(s, rt.dtype)
         self._rows = {}
 
     def _row_numbers(self, n: int, device):
@@ -216,7 +227,7 @@ class RoutedExperts(FeedForward):
             in_eager_step = getattr(ctx, "host_tokens", None) is not None
             if in_eager_step and self.can_group and n * s.top >= GROUP_FROM:
                 self._grouped(x, chosen, weight, h)
-            elif self.fused and n * s.top >= DENSE_FROM * s.n_experts:
+            elif self.fused and n * s.top >= self.dense_from:
                 K.experts_dense(x, rows, chosen, self.gate_up, self.down, h, self.act, 1.0, pair_w=weight, weight_in=self.weight_in)
             else:
                 K.experts_few(x, rows, chosen, self.gate_up, self.row_stride, self.up_off, self.down, h, self.act, 1.0,

@@ -19,6 +19,8 @@ from .norm import LayerNorm
 
 @BLOCKS.register("postnorm")
 class PostNormBlock(Block):
+    reads_stream = True                 # its first sublayer reads the stream in the storage dtype (``CastStream``)
+
     @classmethod
     def declare(cls, spec, prefix=None):
         p = spec.prefix

@@ -16,6 +16,8 @@ from .norm import GroupedRMSNorm
 
 @BLOCKS.register("sum_norm")
 class SumNormBlock(Block):
+    reads_stream = True                 # its first sublayer reads the stream in the storage dtype (``CastStream``)
+
     @classmethod
     def declare(cls, spec, prefix=None):
         p = spec.prefix

@@ -347,6 +347,32 @@ def test_experts_weighed_at_their_input_in_steps_of_every_size(dtype, variant):
             assert _close_rows(got, plain.experts_ff(x.double(), w64, "F.", c), dtype)
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("weight_on", ["input", "output"])
+@pytest.mark.parametrize("hidden,ff,E,top", [(32, 24, 6, 3), (264, 776, 5, 4), (20, 12, 3, 1), (1032, 520, 4, 2)])
+def test_every_way_a_step_of_few_tokens_runs_its_experts(dtype, weight_on, hidden, ff, E, top):
+    """The same step pair by pair, expert by expert and every expert over all tokens, whatever the step would take by
+    itself; rows of lengths that are whole and not whole multiples of a warp's pieces."""
+    spec = _moe_spec(hidden=hidden, intermediate=ff, n_experts=E, top=top, shared=None, weight_on=weight_on)
+    rt = _rt(dtype)
+    cls = FEED_FORWARDS.get(spec.kind)
+    w = random_weights(cls.declare(spec, "F."), 12, 2.0 * hidden ** -0.5, dtype=DT[dtype], device="cuda")
+    part = cls(spec, w, "F.", rt)
+    w64 = _w64(w)
+    c = dict(kind="moe", expert=dict(ff=ff), router=dict(experts=E, top=top))
+    for n in (1, 21):
+        x = torch.randn(n, hidden, generator=torch.Generator().manual_seed(n)).to(DT[dtype])
+        chosen, weight = part.route(x.cuda())
+        if weight_on == "input":
+            want = plain.experts_ff(x.double(), w64, "F.", c, chosen.cpu())
+        else:
+            want = torch.stack([sum(weight[t, k].double().cpu() * plain.gated_ff(x.double()[t:t + 1], w64, f"F.e{int(chosen[t, k])}.")[0]
+                                    for k in range(top)) for t in range(n)])
+        for dense_from, major_from in ((1 << 30, 1 << 30), (1 << 30, 0), (0, 0)):
+            part.dense_from, rt.kernels.EXPERT_MAJOR_FROM = dense_from, major_from
+            assert _close(part.forward(x.cuda(), _ctx([0], [0], [n])).sum(0), want, dtype), f"{n} tokens, {dense_from}, {major_from}"
+
+
 def test_the_products_epilogue_takes_a_factor_per_row():
     """The gated product with a factor per row, in every kernel it may run on (few tokens, many): gate and up times the
     factor before the activation; factors of 1 change no bit."""
