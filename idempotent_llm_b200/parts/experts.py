@@ -26,9 +26,10 @@ GROUP_FROM = 256
 # steps that cannot group (their token ids, or choices, are on the device only) with at least this many (token, choice)
 # pairs per expert run every expert over all tokens with the library's matrix products.  A pair that streams its expert pays
 # for the bytes, an expert's two products for their launches: experts of 5 MB break even at about 13 pairs each (16 of
-# them, 128 pairs: 99 us against 161 us; 256 pairs: 185 us against 169 us), experts of 75 MB at about 3.
+# them, 128 pairs: 99 us against 161 us; 256 pairs: 185 us against 169 us), experts of 75 MB at about 2
+# inside a captured step (8 sequences, 36 layers: 19.7 ms against 19.0 ms a step).
 DENSE_FROM = 12
-LARGE_EXPERT, DENSE_FROM_LARGE = 16 << 20, 3
+LARGE_EXPERT, DENSE_FROM_LARGE = 16 << 20, 2
 
 
 def dense_from(spec, dtype) -> float:
