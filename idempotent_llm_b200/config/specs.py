@@ -107,8 +107,8 @@ class LayerNormSpec:
 
 @dataclass(frozen=True)
 class GroupedRMSNormSpec:
-    """Root-mean-square norm in groups: the row is cut into ``groups`` equal parts of neighbours, each part is divided
-    by its own ``sqrt(mean(part^2) + eps)``, then the whole row is multiplied by a weight ``[size]``."""
+    """Root-mean-square norm of each of ``groups`` equal parts of neighbours of a row: ``v / sqrt(mean(v^2) + eps)`` part by
+    part, then the row times a weight ``[size]``."""
 
     size: int
     eps: float
@@ -391,8 +391,9 @@ class HeadAttentionSpec:
     value_dim, hidden]); ``qk_norm_over`` ``"projection"``: q and k are normed over all their heads' rows at once, with
     weights of that size, before they are split into heads; ``value_norm``: every value head is divided by its root mean
     square (``eps``, no weight) and cached so; ``chunk`` of C: a query at p sees only keys of its own chunk, p - p mod C
-    .. p, chunks counted from the sequence's start; ``weights`` ``"sigmoid"``: no softmax, the weight of a visible key is
-    ``sigmoid(score + z_h)`` with a learned number per head (tensor ``names.score_bias`` [n_heads])."""
+    .. p, chunks counted from the sequence's start; ``weights`` ``"sigmoid"``:
+    keys are weighed by ``sigmoid(score + z_h)``, without a denominator, with a learned number per head (tensor
+    ``names.score_bias`` [n_heads])."""
 
     hidden: int
     n_heads: int

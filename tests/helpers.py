@@ -587,7 +587,7 @@ TOSODRA = {
                                  tosodra_attention(heads=2, kv_heads=2, dim=128, vdim=128, scale=0.09, chunk=700, rot_dims=128, mlp=None),
                                  tosodra_latent(heads=4, dim=48, rot_dim=16, vdim=64, kv_rank=64, scale=0.125,
                                                 mlp=tosodra_moe(experts=20, top=1, ff=64, shared=32)),
-                                 tosodra_attention(heads=8, kv_heads=4, dim=64, vdim=64, scale=0.12, chunk=150, rot_dims=64)],
+                                 tosodra_attention(heads=6, kv_heads=3, dim=64, vdim=64, scale=0.12, chunk=150, rot_dims=64)],
                                 vocab=211, width=96, groups=3, alpha=2.2, emb_scale=7.0),
 }
 
