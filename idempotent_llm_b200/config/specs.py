@@ -85,11 +85,13 @@ class DyTNormSpec:
 @dataclass(frozen=True)
 class NormSpec:
     """Root-mean-square norm over the last axis, weight applied afterwards.
-    ``weight``: the tensor's name behind the prefix the block gives the norm."""
+    ``weight``: the tensor's name behind the prefix the block gives the norm.  ``weight_offset`` is added to the stored
+    weight (1: the tensor holds what is added to one)."""
 
     size: int
     eps: float
     weight: str = "weight"
+    weight_offset: float = 0.0
     kind: str = "rmsnorm"
 
 
@@ -168,12 +170,16 @@ class AttentionSpec:
 @dataclass(frozen=True)
 class GatedMLPSpec:
     """Dense gated feed-forward: ``down(act(gate(x)) * up(x))``
-    (reference: src/detllm/model.py:415-427, src/detllm/ops/di_swiglu.py:43-45)."""
+    (reference: src/detllm/model.py:415-427, src/detllm/ops/di_swiglu.py:43-45).  ``activation`` ``"clamped"`` bounds both
+    branches: with ``g = min(gate(x), limit)`` and ``u = clamp(up(x), -limit, limit)`` it is ``down(g * sigmoid(slope g) * (u +
+    1))``."""
 
     hidden: int
     intermediate: int
     names: GatedMLPNames
     activation: str = "silu"
+    limit: float = 0.0
+    slope: float = 0.0
     kind: str = "gated_mlp"
 
 
@@ -188,6 +194,7 @@ class LatentAttentionNames:
     up_v: str = "uv"
     o: str = "o"
     sink: str = "sink"
+    gate: str = "g"
 
 
 @dataclass(frozen=True)
@@ -200,7 +207,9 @@ class LatentAttentionSpec:
     all heads share.  Head h's unrotated key is ``Uk_h c`` and its value ``Uv_h c`` (``value_dim`` numbers); the score
     is ``(q_plain . k_plain + q_rot . k_rot) * softmax_scale``.  ``position`` (variant ``"interleaved"`` or
     ``"half_partial"``) turns the first ``position.dim`` of the rotated dims.  ``sink``: one learned score per head joins the softmax's
-    denominator with no key and no value.  Only ``c`` and the rotated key part are kept per token."""
+    denominator with no key and no value.  Only ``c`` and the rotated key part are kept per token.  ``rot_dim`` may be 0
+    (attention without positions).  ``window`` of W: a query at p sees positions p - W + 1 .. p.  ``gate``: the merged heads
+    times the sigmoid of a projection of the mixer's input (tensor ``names.gate`` [n_heads * value_dim, hidden])."""
 
     hidden: int
     n_heads: int
@@ -212,6 +221,8 @@ class LatentAttentionSpec:
     eps: float
     position: Optional[RotarySpec] = None
     sink: bool = False
+    window: Optional[int] = None
+    gate: bool = False
     names: LatentAttentionNames = LatentAttentionNames()
     kind: str = "latent_attention"
 
@@ -264,7 +275,9 @@ class RoutedExpertsSpec:
 
     ``scores`` ``"sigmoid"``: ``s = sigmoid(z)`` element by element instead of the softmax.  ``correction`` None: experts are
     chosen by ``s`` itself.  ``renormalize`` False: the weights are the chosen ``s`` times ``scale`` as they are.
-    ``weight_on`` ``"input"``: a weight multiplies its expert's input instead of its output, ``expert(w x)``."""
+    ``weight_on`` ``"input"``: a weight multiplies its expert's input instead of its output, ``expert(w x)``.  ``group_top``: a
+    group's score is the sum of its so many largest choice scores.  ``shared_gate`` (a tensor ``[1, hidden]``): the shared
+    expert's output is multiplied by the sigmoid of that projection of the token, a number per token."""
 
     hidden: int
     intermediate: int
@@ -281,6 +294,8 @@ class RoutedExpertsSpec:
     scores: str = "softmax"
     renormalize: bool = True
     weight_on: str = "output"
+    group_top: int = 1
+    shared_gate: Optional[str] = None
     expert: str = "e{}."
     names: GatedMLPNames = GatedMLPNames(gate="gate", up="up", down="down")
     kind: str = "routed_experts"
@@ -321,6 +336,77 @@ class SinkAttentionSpec:
     gate: bool = True
     names: SinkAttentionNames = SinkAttentionNames()
     kind: str = "sink_attention"
+
+
+@dataclass(frozen=True)
+class DifferentialAttentionNames:
+    """Checkpoint names of a differential attention's tensors, behind the mixer's prefix; a filter's tensor is its
+    projection's name plus ``conv``."""
+
+    q: str = "q"
+    k: str = "k"
+    v: str = "v"
+    o: str = "o"
+    gate: str = "g"
+    conv: str = ".conv"
+    lambda_q1: str = "lq1"
+    lambda_k1: str = "lk1"
+    lambda_q2: str = "lq2"
+    lambda_k2: str = "lk2"
+
+
+@dataclass(frozen=True)
+class DifferentialAttentionSpec:
+    """Causal grouped-query attention (a *mixer*) whose heads have two maps and one set of values.  A q or k head is ``[map 1, map
+    2]``, ``key_dim`` dims each; q, k and v channels pass a causal filter over time of ``conv_taps`` taps directly behind the
+    projections (None: no filter; one tap is a factor), then the first ``position.dim`` dims of each map are turned
+    (variant ``"half_partial"``).  Each map is a softmax attention of its own with scores ``q . k * softmax_scale``; with
+    their contexts a1, a2 and ``lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff`` a head goes on as ``o = a1 - lambda a2``, over
+    its root mean square over ``value_dim`` (``eps``), times ``1 - diff``.  ``head_gate``: times the sigmoid of one number per
+    head projected from the mixer's input."""
+
+    hidden: int
+    n_heads: int
+    n_kv_heads: int
+    key_dim: int                    # of one map
+    value_dim: int
+    softmax_scale: float
+    diff: float
+    eps: float
+    conv_taps: Optional[int] = None
+    position: Optional[RotarySpec] = None
+    head_gate: bool = True
+    names: DifferentialAttentionNames = DifferentialAttentionNames()
+    kind: str = "differential_attention"
+
+
+@dataclass(frozen=True)
+class RetentionNames:
+    """Checkpoint names of a retention's tensors, behind the mixer's prefix."""
+
+    q: str = "q"
+    k: str = "k"
+    v: str = "v"
+    gate: str = "g"
+    o: str = "o"
+
+
+@dataclass(frozen=True)
+class RetentionSpec:
+    """A linear recurrence whose heads fade at constant rates (a *mixer*): q and k (``heads`` of ``key_dim``) turned over the
+    first ``position.dim`` dims of each head (variant ``"half_partial"``), k then times ``key_dim ** -0.5``; per head ``S <-
+    decay_h S + k v^T``, ``o = S^T q``; each head's read-out over its root mean square (``eps``, no weight), the merged heads
+    times ``silu`` of a full projection of the mixer's input, then the output projection."""
+
+    hidden: int
+    heads: int
+    key_dim: int
+    value_dim: int
+    decay: Tuple[float, ...]
+    eps: float
+    position: Optional[RotarySpec] = None
+    names: RetentionNames = RetentionNames()
+    kind: str = "retention"
 
 
 @dataclass(frozen=True)

@@ -152,6 +152,21 @@ __device__ __forceinline__ float gelu_tanh_f(float g) {
 __device__ __forceinline__ float gated_act(float g, float u, int act) {
     return act == 1 ? gelu_tanh_f(g) * u : act == 2 ? fmaxf(g, 0.f) * u : silu_mul(g, u);
 }
+// act 3, with two constants: the gate clamped from above and the up branch from both sides, g = min(g, limit), u =
+// clamp(u, -limit, limit), then g * sigmoid(slope g) * (u + 1)
+#define IDM_ACT_CLAMPED 3
+__device__ __forceinline__ float clamped_act(float g, float u, float limit, float slope) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+#if defined(IDM_F32)
+    return g / (1.0f + expf(-slope * g)) * (u + 1.0f);
+#else
+    return __fmul_rn(__fdividef(g, 1.0f + __expf(-slope * g)), u + 1.0f);
+#endif
+}
+__device__ __forceinline__ float gated_act(float g, float u, int act, float limit, float slope) {
+    return act == IDM_ACT_CLAMPED ? clamped_act(g, u, limit, slope) : gated_act(g, u, act);
+}
 
 // ------------------------------------------------------------ reductions
 // Fixed-order reductions: xor butterflies inside a warp, then the warps' values

@@ -683,8 +683,8 @@ extern "C" int idm_delta_scan(const float* c, int c_stride, int c_q, int c_k, in
 }
 
 // ------------------------------------------------------------------ behind the recurrence
-// out[t, out_col + h dv + j] = o[t, h, j] / sqrt(mean_j o^2 + eps) * w[j] * act(gate[t, gate_col + h dv + j]) * scale,
-// act = sigmoid (gate_act 0) or silu (gate_act 1); one warp per (token, head)
+// out[t, out_col + h dv + j] = o[t, h, j] / sqrt(mean_j o^2 + eps) * w[j] * act(gate[t, gate_col + h dv + j]) * scale (w
+// null: ones), act = sigmoid (gate_act 0) or silu (gate_act 1); one warp per (token, head)
 __global__ void __launch_bounds__(128) delta_out_kernel(const float* __restrict__ o, int o_stride, const float* __restrict__ w,
                                                         float eps, const float* __restrict__ gate, int gate_stride,
                                                         int gate_col, int gate_act, float scale, T* __restrict__ out,
@@ -703,7 +703,8 @@ __global__ void __launch_bounds__(128) delta_out_kernel(const float* __restrict_
     T* dst = out + (size_t)t * out_stride + out_col + (size_t)h * dv;
     for (int d = lane; d < dv; d += 32) {
         const float z = gr[d], sg = 1.0f / (1.0f + expf(-z));
-        from_f32(dst[d], gate_act == 1 ? x[d] * inv * w[d] * (z * sg) * scale : x[d] * inv * w[d] / (1.0f + expf(-z)) * scale);
+        const float y = w ? x[d] * inv * w[d] : x[d] * inv;
+        from_f32(dst[d], gate_act == 1 ? y * (z * sg) * scale : y / (1.0f + expf(-z)) * scale);
     }
 }
 

@@ -625,11 +625,13 @@ extern "C" int idm_post_pre_norm(float* h, const float* y, const float* w_post, 
 }
 
 // ------------------------------------------------------ gated activations, by name
-// (gated_act in common.cuh: act 0 is g * sigmoid(g) * u, act 1 the tanh form of gelu times u)
+// (gated_act in common.cuh: act 0 is g * sigmoid(g) * u, act 1 the tanh form of gelu times u, act 2 relu times u, act 3 the
+// clamped form with its two constants)
 
 // y[t, i] = act(gu[t, i]) * gu[t, inter + i] of a 32-bit gate/up product [N, 2 * inter]
 __global__ void __launch_bounds__(256) gated_act_kernel(const float* __restrict__ gu, T* __restrict__ y, int inter, int act,
-                                                        const float* __restrict__ row_w) {
+                                                        float limit, float slope, const float* __restrict__ row_w,
+                                                        const float* __restrict__ row_out) {
     pdl_launch_dependents();
     pdl_wait();
     const int c = blockIdx.y * blockDim.x + threadIdx.x;
@@ -637,13 +639,16 @@ __global__ void __launch_bounds__(256) gated_act_kernel(const float* __restrict_
     const size_t t = blockIdx.x;
     float g = gu[t * 2 * (size_t)inter + c], u = gu[t * 2 * (size_t)inter + inter + c];
     if (row_w) { g *= row_w[t]; u *= row_w[t]; }                 // a factor on the row's input (gate and up are linear)
-    from_f32(y[t * (size_t)inter + c], gated_act(g, u, act));
+    const float v = gated_act(g, u, act, limit, slope);
+    from_f32(y[t * (size_t)inter + c], row_out ? v * row_out[t] : v);      // a factor on what the activation gives
 }
 
-extern "C" int idm_gated_act(const float* gu, void* y, int n_tokens, int inter, int act, const float* row_w, cudaStream_t stream) {
+extern "C" int idm_gated_act(const float* gu, void* y, int n_tokens, int inter, int act, float limit, float slope,
+                             const float* row_w, const float* row_out, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
-    IDM_REQUIRE(inter > 0 && act >= 0 && act <= 2, "gated_act: inter=%d act=%d", inter, act);
-    idm_launch(gated_act_kernel, dim3(n_tokens, (inter + 255) / 256), dim3(256), 0, stream, gu, (T*)y, inter, act, row_w);
+    IDM_REQUIRE(inter > 0 && act >= 0 && act <= IDM_ACT_CLAMPED, "gated_act: inter=%d act=%d", inter, act);
+    idm_launch(gated_act_kernel, dim3(n_tokens, (inter + 255) / 256), dim3(256), 0, stream, gu, (T*)y, inter, act, limit, slope, row_w,
+               row_out);
     IDM_LAUNCH_CHECK("gated_act");
     return 0;
 }
@@ -675,34 +680,38 @@ extern "C" int idm_token_gate(const float* s, const int* tokens, const void* tab
 
 // ------------------------------------------------------------- output gate of a mixer
 // out[t, out_col + c] = o[t, c] * sigmoid(gate[t * gate_stride + c]) * scale   (gate null: only the constant);
-// o [N, width] in the storage type, gate 32-bit (columns of a wider projection), out rows of out_stride.
+// o [N, width] in the storage type, gate 32-bit (columns of a wider projection), out rows of out_stride.  Heads of `in_head`
+// elements in o of which the first `out_head` count (padded heads): out and gate hold those alone.
 __global__ void __launch_bounds__(256) gate_scale_kernel(const T* __restrict__ o, const float* __restrict__ gate,
                                                          int gate_stride, int gate_group, float scale, T* __restrict__ out,
-                                                         int out_stride, int out_col, int width) {
+                                                         int out_stride, int out_col, int width, int in_head, int out_head) {
     pdl_launch_dependents();
     pdl_wait();
     const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
     if (c >= width) return;
     const size_t t = blockIdx.x;
-    const T* src = o + t * width + c;
+    const T* src = o + t * (size_t)(width / out_head * in_head);
     T* dst = out + t * out_stride + out_col + c;
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
         if (c + i >= width) break;
-        float v = to_f32(src[i]);
+        const int ci = c + i;
+        float v = to_f32(src[in_head == out_head ? ci : ci / out_head * in_head + ci % out_head]);
         if (gate) v = v / (1.0f + expf(-gate[t * gate_stride + (c + i) / gate_group]));
         from_f32(dst[i], v * scale);
     }
 }
 
 extern "C" int idm_gate_scale(const void* o, const float* gate, int gate_stride, int gate_group, float scale, void* out,
-                              int out_stride, int out_col, int n_tokens, int width, cudaStream_t stream) {
+                              int out_stride, int out_col, int n_tokens, int width, int in_head, int out_head, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
     IDM_REQUIRE(width > 0 && out_col >= 0 && out_col + width <= out_stride, "gate_scale: columns %d..%d of rows of %d", out_col,
                 out_col + width, out_stride);
     IDM_REQUIRE(gate_group >= 1, "gate_scale: a gate serves %d columns", gate_group);
+    IDM_REQUIRE(out_head >= 1 && in_head >= out_head && width % out_head == 0, "gate_scale: %d of %d elements of a head, %d columns",
+                out_head, in_head, width);
     idm_launch(gate_scale_kernel, dim3(n_tokens, (width + 1023) / 1024), dim3(256), 0, stream, (const T*)o, gate, gate_stride,
-               gate_group, scale, (T*)out, out_stride, out_col, width);
+               gate_group, scale, (T*)out, out_stride, out_col, width, in_head, out_head);
     IDM_LAUNCH_CHECK("gate_scale");
     return 0;
 }

@@ -99,9 +99,17 @@ struct GemmEpi {
     float* out;          // STORE: [M, N]; RESIDUAL: the residual stream [M, N]
     T* y; int inter;     // SWIGLU: y [M, inter]
     int act;             // SWIGLU: which gated activation (gated_act in common.cuh; 0 = silu)
+    float limit, slope;  // SWIGLU: the constants of the clamped activation
     const float* row_w;  // SWIGLU, or null: row_w[t] multiplies gate and up of token t before the activation
+    const float* row_out;    // SWIGLU, or null: row_out[t] multiplies what the activation gives
     QkvArgs q;           // QKV
 };
+
+// four features of the gated activation from (gate, up) pairs side by side
+__device__ __forceinline__ void gated_act4(float* y, float4 a, float4 b, const GemmEpi& e) {
+    y[0] = gated_act(a.x, a.y, e.act, e.limit, e.slope); y[1] = gated_act(a.z, a.w, e.act, e.limit, e.slope);
+    y[2] = gated_act(b.x, b.y, e.act, e.limit, e.slope); y[3] = gated_act(b.z, b.w, e.act, e.limit, e.slope);
+}
 
 // ------------------------------------------------------------------- persistent kernel (many tokens)
 // Above 256 tokens nothing is split and the product is bound by the tensor cores.  One block per SM
@@ -199,8 +207,14 @@ __device__ __forceinline__ void persistent_tile_epilogue(const GemmEpi& e, uint3
                         p0.x *= rw; p0.y *= rw; p0.z *= rw; p0.w *= rw; p1.x *= rw; p1.y *= rw; p1.z *= rw; p1.w *= rw;
                         p2.x *= rw; p2.y *= rw; p2.z *= rw; p2.w *= rw; p3.x *= rw; p3.y *= rw; p3.z *= rw; p3.w *= rw;
                     }
-                    const float y8[8] = {gated_act(p0.x, p0.y, e.act), gated_act(p0.z, p0.w, e.act), gated_act(p1.x, p1.y, e.act), gated_act(p1.z, p1.w, e.act),
-                                         gated_act(p2.x, p2.y, e.act), gated_act(p2.z, p2.w, e.act), gated_act(p3.x, p3.y, e.act), gated_act(p3.z, p3.w, e.act)};
+                    float y8[8];
+                    gated_act4(y8, p0, p1, e);
+                    gated_act4(y8 + 4, p2, p3, e);
+                    if (e.row_out) {
+                        const float ro = e.row_out[t0 + c0 + j];
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) y8[i] = __fmul_rn(y8[i], ro);
+                    }
                     const int fg = tx * 64 + sub * 8;
                     T* dst = e.y + (size_t)(t0 + c0 + j) * e.inter + fg;
                     if ((e.inter & 7) == 0 && fg + 8 <= e.inter) {
@@ -1045,6 +1059,7 @@ __global__ void __launch_bounds__(GS_THREADS) gemm_small_kernel(const __grid_con
                     // the tile's columns are gate, up, gate, up, ... of the features f0 / 2 ..; 32 columns are asked
                     // for before the first is waited for
                     const float rw = e.row_w && live ? e.row_w[t] : 1.0f;      // (a factor of 1 changes no bit)
+                    const float ro = e.row_out && live ? e.row_out[t] : 1.0f;
 #pragma unroll 1
                     for (int c0 = 0; c0 < bf; c0 += 32) {
                         if (((f0 + c0) >> 1) >= e.inter) break;
@@ -1060,7 +1075,8 @@ __global__ void __launch_bounds__(GS_THREADS) gemm_small_kernel(const __grid_con
                             float y8[8];
 #pragma unroll
                             for (int i = 0; i < 8; ++i)
-                                y8[i] = gated_act(__fmul_rn(__uint_as_float(raw[16 * h + 2 * i]), rw), __fmul_rn(__uint_as_float(raw[16 * h + 2 * i + 1]), rw), e.act);
+                                y8[i] = __fmul_rn(gated_act(__fmul_rn(__uint_as_float(raw[16 * h + 2 * i]), rw), __fmul_rn(__uint_as_float(raw[16 * h + 2 * i + 1]), rw), e.act,
+                                                            e.limit, e.slope), ro);
                             T* dst = e.y + (size_t)t * e.inter + fg;
                             if ((e.inter & 7) == 0 && fg + 8 <= e.inter) {
                                 store8(dst, y8);
@@ -1451,14 +1467,21 @@ extern "C" int idm_gemm_bf16_swiglu(const void* x, const void* w_tiled, void* y,
 }
 
 // the same product with the gated activation chosen by number (gated_act in common.cuh): y = act(x . gate^T) * (x . up^T)
-// with, if given, a factor per row: y[t] = act(row_w[t] x_t . gate^T) * (row_w[t] x_t . up^T)
-extern "C" int idm_gemm_bf16_gated_rows(const void* x, const void* w_tiled, void* y, int M, int inter, int K, int act,
-                                        const float* row_w, cudaStream_t stream) {
-    IDM_REQUIRE(act >= 0 && act <= 2, "gemm_gated: activation %d is not built", act);
+// with, if given, a factor per row on the input, act(row_w[t] x_t . gate^T) * (row_w[t] x_t . up^T), and one on the
+// result, y[t] = row_out[t] * (...); `limit` and `slope` are the constants of the clamped activation (act 3)
+extern "C" int idm_gemm_bf16_gated_all(const void* x, const void* w_tiled, void* y, int M, int inter, int K, int act,
+                                       float limit, float slope, const float* row_w, const float* row_out, cudaStream_t stream) {
+    IDM_REQUIRE(act >= 0 && act <= IDM_ACT_CLAMPED, "gemm_gated: activation %d is not built", act);
     GemmEpi e = {};
-    e.y = (T*)y; e.inter = inter; e.act = act; e.row_w = row_w;
+    e.y = (T*)y; e.inter = inter; e.act = act; e.row_w = row_w; e.row_out = row_out; e.limit = limit; e.slope = slope;
     const int tiles = (inter + 63) / 64;
     return gemm_any<EPI_SWIGLU>(x, w_tiled, e, M, tiles * GT_BM, K, stream);
+}
+
+extern "C" int idm_gemm_bf16_gated_rows(const void* x, const void* w_tiled, void* y, int M, int inter, int K, int act,
+                                        const float* row_w, cudaStream_t stream) {
+    IDM_REQUIRE(act >= 0 && act < IDM_ACT_CLAMPED, "gemm_gated: activation %d takes constants or is not built", act);
+    return idm_gemm_bf16_gated_all(x, w_tiled, y, M, inter, K, act, 0.f, 0.f, row_w, nullptr, stream);
 }
 
 extern "C" int idm_gemm_bf16_gated(const void* x, const void* w_tiled, void* y, int M, int inter, int K, int act,

@@ -82,7 +82,8 @@ extern "C" int idm_latent_kv_finish(const float* proj, int ld, int col0, int R, 
 // eight warps each take an eighth of the i (a lane owns an output and reads W side by side with its neighbours),
 // and the eight partial sums of an element are added in ascending order, so the order of every sum depends on I
 // alone.  `tail` more columns of x behind the I are copied behind the O outputs, the first `rot_dims` of them
-// turned by the token's angles (a query's rotated part).  A head's matrix is read once per HW_TOKENS tokens.
+// turned by the token's angles (a query's rotated part).  A head's matrix is read once per HW_TOKENS tokens.  With `gate` (32-bit
+// rows of stride gate_stride, columns h * O + o) an output is multiplied by the sigmoid of its gate before it is rounded.
 #define HW_TOKENS 8
 #define HW_WARPS 8          // (warp w also adds token w's partial sums: as many warps as tokens)
 static_assert(HW_WARPS == HW_TOKENS, "a warp per token in the last phase");
@@ -91,7 +92,8 @@ template <typename OutT>
 __global__ void __launch_bounds__(HW_WARPS * 32) headwise_kernel(const float* __restrict__ x, long long x_tok, int x_head, int I,
                                                                  const T* __restrict__ W, int O, OutT* __restrict__ out,
                                                                  long long o_tok, int o_head, int tail, int rot_dims, int halves,
-                                                                 const float2* __restrict__ cs, int half, float mag, int n_tokens) {
+                                                                 const float2* __restrict__ cs, int half, float mag,
+                                                                 const float* __restrict__ gate, int gate_stride, int n_tokens) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ float xs[];                       // [HW_TOKENS][I], then the warps' partial sums [HW_WARPS][HW_TOKENS][32]
@@ -126,7 +128,10 @@ __global__ void __launch_bounds__(HW_WARPS * 32) headwise_kernel(const float* __
         float s = 0.f;
 #pragma unroll
         for (int w = 0; w < HW_WARPS; ++w) s += part[(w * HW_TOKENS + tt) * 32 + lane];
-        if (tt < nt && o < O) from_f32(out[(size_t)(t0 + tt) * o_tok + (size_t)h * o_head + o], s);
+        if (tt < nt && o < O) {
+            if (gate) s = s / (1.0f + expf(-gate[(size_t)(t0 + tt) * gate_stride + h * O + o]));
+            from_f32(out[(size_t)(t0 + tt) * o_tok + (size_t)h * o_head + o], s);
+        }
     }
     if (blockIdx.z != 0) return;
     for (int e = threadIdx.x; e < nt * tail; e += blockDim.x) {
@@ -139,23 +144,24 @@ __global__ void __launch_bounds__(HW_WARPS * 32) headwise_kernel(const float* __
 // out_is_f32: the outputs are 32-bit (queries in the latent's space); else the storage type (a product's input)
 extern "C" int idm_headwise(const float* x, long long x_tok, int x_head, int I, const void* W, int O, void* out,
                             int out_is_f32, long long o_tok, int o_head, int tail, int rot_dims, int halves, const float* cs, int half,
-                            float mag, int n_tokens, int n_heads, cudaStream_t stream) {
+                            float mag, const float* gate, int gate_stride, int n_tokens, int n_heads, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
     IDM_REQUIRE(I > 0 && O >= 0 && n_heads > 0 && tail >= 0, "headwise: sizes I=%d O=%d heads=%d tail=%d", I, O, n_heads, tail);
     IDM_REQUIRE(rot_dims >= 0 && rot_dims <= tail && rot_dims % 2 == 0 && (rot_dims == 0 || (cs != nullptr && half >= rot_dims / 2)),
                 "headwise: %d turned dims of %d with a table of %d angles", rot_dims, tail, half);
     const size_t smem = ((size_t)HW_TOKENS * I + HW_WARPS * HW_TOKENS * 32) * sizeof(float);
     IDM_REQUIRE(smem <= 200 * 1024, "headwise: I=%d does not fit shared memory", I);
+    IDM_REQUIRE(gate == nullptr || gate_stride >= n_heads * O, "headwise: gates of %d x %d in rows of %d", n_heads, O, gate_stride);
     const dim3 grid((n_tokens + HW_TOKENS - 1) / HW_TOKENS, n_heads, max(1, (O + 31) / 32));
     IDM_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "headwise: %d heads, %d outputs", n_heads, O);
     if (out_is_f32) {
         if (smem > 48 * 1024) cudaFuncSetAttribute(headwise_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         idm_launch(headwise_kernel<float>, grid, dim3(HW_WARPS * 32), smem, stream, x, x_tok, x_head, I, (const T*)W, O, (float*)out,
-                   o_tok, o_head, tail, rot_dims, halves, (const float2*)cs, half, mag, n_tokens);
+                   o_tok, o_head, tail, rot_dims, halves, (const float2*)cs, half, mag, gate, gate_stride, n_tokens);
     } else {
         if (smem > 48 * 1024) cudaFuncSetAttribute(headwise_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         idm_launch(headwise_kernel<T>, grid, dim3(HW_WARPS * 32), smem, stream, x, x_tok, x_head, I, (const T*)W, O, (T*)out,
-                   o_tok, o_head, tail, rot_dims, halves, (const float2*)cs, half, mag, n_tokens);
+                   o_tok, o_head, tail, rot_dims, halves, (const float2*)cs, half, mag, gate, gate_stride, n_tokens);
     }
     IDM_LAUNCH_CHECK("headwise");
     return 0;
@@ -168,7 +174,8 @@ extern "C" int idm_headwise(const float* x, long long x_tok, int x_head, int I, 
 // positions, staged in shared memory once for all the block's heads (two buffers: the next block's copies run
 // while this one is scored); lane i scores key j0 + i against the head's
 // query (kept in shared memory, 32-bit), the running (max, sum, context) is rescaled block by block, and the
-// context is a weighted sum of the rows' first R numbers, a lane owning pairs of neighbours.  With one run the
+// context is a weighted sum of the rows' first R numbers, a lane owning pairs of neighbours.  With a window a query walks from
+// its first key on.  With one run the
 // block finishes the row (the sink, a score with no key and no value, joins the sum once) and writes the context
 // [N, H, R] in 32-bit; with several, every run leaves (max, sum, context) in scratch and latent_fold_kernel adds
 // the runs in ascending order.
@@ -185,7 +192,17 @@ struct LatentArgs {
     int n_tokens, H, R, D;
     float scale;
     int run_keys, n_runs, stride_words, n_buf;
+    int window;               // > 0: a query at p sees keys p - window + 1 .. p; 0: every earlier key
 };
+
+// keys lo .. hi of run `run` of a query at `pos` (lo > pos: none).  Runs lie at absolute positions; with a window a
+// query's run 0 is the one that holds its first key.
+__device__ __forceinline__ void latent_run(const LatentArgs& a, int pos, int run, int& lo, int& hi) {
+    const int first = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+    const int at = (first / a.run_keys + run) * a.run_keys;
+    lo = max(at, first);
+    hi = min(pos, at + a.run_keys - 1);
+}
 
 template <int NACC, int HPW>
 __global__ void __launch_bounds__(LA_WARPS * 32) latent_attention_kernel(LatentArgs a) {
@@ -201,7 +218,8 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attention_kernel(LatentA
     const bool live_head = head < a.H;
     const int nh = min(HPW, a.H - head);                                      // (heads of this warp that exist)
     const int pos = a.positions[t], slot = a.slots[a.token_seq[t]];
-    const int lo = run * a.run_keys, hi = min(pos, lo + a.run_keys - 1);      // keys lo .. hi
+    int lo, hi;
+    latent_run(a, pos, run, lo, hi);                                          // keys lo .. hi
     float m[HPW], l[HPW];
     float acc[HPW][NACC];
 #pragma unroll
@@ -406,7 +424,8 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_attention_mma_kernel(Lat
     const int t = blockIdx.x, head0 = blockIdx.y * 16, run = blockIdx.z;
     const int nh = min(16, a.H - head0);
     const int pos = a.positions[t], slot = a.slots[a.token_seq[t]];
-    const int lo = run * a.run_keys, hi = min(pos, lo + a.run_keys - 1);
+    int lo, hi;
+    latent_run(a, pos, run, lo, hi);
     const int NT = a.R / 32;                                                  // 8-column tiles of the context a warp owns
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};                   // rows g and g + 8
     float o[NT_MAX][4];
@@ -542,7 +561,7 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_attention_mma_kernel(Lat
 #define LF_THREADS 256
 __global__ void __launch_bounds__(LF_THREADS) latent_fold_kernel(const float* __restrict__ part, const float* __restrict__ sink,
                                                                  float* __restrict__ ctx, const int* __restrict__ positions,
-                                                                 int n_tokens, int H, int R, int run_keys, int n_runs) {
+                                                                 int n_tokens, int H, int R, int run_keys, int n_runs, int window) {
     pdl_launch_dependents();
     pdl_wait();
     __shared__ float wts[LF_MAX_RUNS];
@@ -550,7 +569,8 @@ __global__ void __launch_bounds__(LF_THREADS) latent_fold_kernel(const float* __
     const int lane = threadIdx.x & 31;
     const long long w = blockIdx.x;
     const int t = (int)(w / H), head = (int)(w % H);
-    const int used = min(n_runs, positions[t] / run_keys + 1);               // runs that hold keys of this query
+    const int pos = positions[t], first = window > 0 ? max(0, pos - window + 1) : 0;
+    const int used = min(n_runs, pos / run_keys - first / run_keys + 1);     // runs that hold keys of this query
     const size_t stride = (size_t)R + 2;
     const float* p = part + (size_t)w * n_runs * stride;
     if (threadIdx.x < 32) {
@@ -603,11 +623,12 @@ extern "C" int idm_latent_attention_heads_per_block(int H, int R, int D) {
     return latent_mma_fits(R, D) ? 16 : (H > LA_WARPS ? 2 * LA_WARPS : LA_WARPS);
 }
 
-// run_keys: a multiple of 32; n_runs * run_keys covers every position of the step (n_runs == 1: no scratch)
+// run_keys: a multiple of 32; n_runs * run_keys covers every position of the step, or with a window every key from any
+// query's first key's run on (n_runs == 1: no scratch; with a window run_keys then exceeds every position)
 extern "C" int idm_latent_attention(const float* qa, const void* pool, const int* table, int table_stride,
                                     const int* token_seq, const int* positions, const int* slots, const float* sink,
                                     float* ctx, float* part, int n_tokens, int H, int R, int D, float scale,
-                                    int run_keys, int n_runs, cudaStream_t stream) {
+                                    int run_keys, int n_runs, int window, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
     IDM_REQUIRE(H > 0 && R > 0 && D >= R && R <= 1024, "latent_attention: heads=%d rank=%d row=%d (rank at most 1024)", H, R, D);
     IDM_REQUIRE(n_runs >= 1 && n_runs <= LF_MAX_RUNS && run_keys > 0 && run_keys % 32 == 0 && (n_runs == 1 || part != nullptr),
@@ -616,6 +637,7 @@ extern "C" int idm_latent_attention(const float* qa, const void* pool, const int
     a.qa = qa; a.pool = (const T*)pool; a.table = table; a.table_stride = table_stride;
     a.token_seq = token_seq; a.positions = positions; a.slots = slots; a.sink = sink; a.ctx = ctx; a.part = part;
     a.n_tokens = n_tokens; a.H = H; a.R = R; a.D = D; a.scale = scale; a.run_keys = run_keys; a.n_runs = n_runs;
+    a.window = window > 0 ? window : 0;
 #if defined(IDM_BF16)
     if (idm_latent_attention_heads_per_block(H, R, D) == 16 && latent_mma_fits(R, D)) {
         int units = D / 8;                                  // rows of 16 bytes x an odd number: no bank is hit twice by a fragment load
@@ -638,7 +660,7 @@ extern "C" int idm_latent_attention(const float* qa, const void* pool, const int
         IDM_LAUNCH_CHECK("latent_attention_mma");
         if (n_runs > 1) {
             idm_launch(latent_fold_kernel, dim3((unsigned)(n_tokens * H)), dim3(LF_THREADS), 0, stream, (const float*)part, sink, ctx,
-                       positions, n_tokens, H, R, run_keys, n_runs);
+                       positions, n_tokens, H, R, run_keys, n_runs, a.window);
             IDM_LAUNCH_CHECK("latent_fold");
         }
         return 0;
@@ -675,7 +697,7 @@ extern "C" int idm_latent_attention(const float* qa, const void* pool, const int
     IDM_LAUNCH_CHECK("latent_attention");
     if (n_runs > 1) {
         idm_launch(latent_fold_kernel, dim3((unsigned)(n_tokens * H)), dim3(LF_THREADS), 0, stream, (const float*)part, sink, ctx,
-                   positions, n_tokens, H, R, run_keys, n_runs);
+                   positions, n_tokens, H, R, run_keys, n_runs, a.window);
         IDM_LAUNCH_CHECK("latent_fold");
     }
     return 0;

@@ -4,10 +4,12 @@
 //   s      = softmax(z) over all E experts, or sigmoid(z) element by element, 32-bit
 //   c_e    = s_e + correction_e                           the score an expert is CHOSEN by (sigmoids without a correction:
 //                                                         z itself, whose order is the same and which does not saturate)
-//   groups : E / count neighbours each; a group's score is its largest c; only experts of the `keep` best groups
-//            can be chosen (the others count as minus infinity)
+//   groups : E / count neighbours each; a group's score is the sum of its `group_top` largest c (1: its largest); only
+//            experts of the `keep` best groups can be chosen (the others count as minus infinity)
 //   chosen : the `top` largest c among those, in descending order (ties: the lower index)
 //   weight : s_chosen / (sum of the chosen s + 1e-20) * scale, or (not renormalized) s_chosen * scale
+//
+// A column behind the E logits may hold a gate's pre-activation (a shared expert's): its sigmoid goes to gate_out[t].
 //
 // One warp per token; s and c wait in shared memory.  Nothing here depends on the other tokens of the step.
 #include "common.cuh"
@@ -27,7 +29,8 @@ __device__ __forceinline__ void warp_argmax(float& v, int& idx) {
 __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const float* __restrict__ z, int z_stride,
                                                               const float* __restrict__ correction, int* __restrict__ chosen,
                                                               float* __restrict__ weight, int n_tokens, int E, int top,
-                                                              int count, int keep, float scale, int sigmoid, int renorm) {
+                                                              int count, int keep, int group_top, float scale, int sigmoid,
+                                                              int renorm, float* __restrict__ gate_out) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ float sm[];
@@ -38,6 +41,7 @@ __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const float* __res
     float* c = s + E;                                            // [E] choice scores (minus infinity once taken or shut out)
     float* gs = c + E;                                           // [count] group scores
     const float* zr = z + (size_t)t * z_stride;
+    if (gate_out && lane == 0) gate_out[t] = 1.0f / (1.0f + expf(-zr[E]));
     if (sigmoid) {
         for (int e = lane; e < E; e += 32) {
             const float v = zr[e];
@@ -59,7 +63,19 @@ __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const float* __res
         for (int g = lane; g < count; g += 32) {
             float best = -INFINITY;
             for (int e = g * per; e < (g + 1) * per; ++e) best = fmaxf(best, c[e]);
-            gs[g] = best;
+            float sum = best, last = best;
+            int at = -1;                                         // where `last` was found (of equal scores: the lowest first)
+            for (int e = g * per; e < (g + 1) * per && at < 0; ++e)
+                if (c[e] == best) at = e;
+            for (int k = 1; k < group_top && k < per; ++k) {     // the next one down: smaller, or equal and further up
+                float v = -INFINITY;
+                int idx = -1;
+                for (int e = g * per; e < (g + 1) * per; ++e)
+                    if ((c[e] < last || (c[e] == last && e > at)) && (idx < 0 || c[e] > v)) { v = c[e]; idx = e; }
+                if (idx < 0) break;
+                sum += v; last = v; at = idx;
+            }
+            gs[g] = sum;
         }
         __syncwarp();
         // the `keep` best groups, one after another; gs of a kept group becomes +infinity as its mark
@@ -95,18 +111,19 @@ __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const float* __res
 }
 
 extern "C" int idm_route(const float* z, int z_stride, const float* correction, int* chosen, float* weight, int n_tokens,
-                         int n_experts, int top, int groups, int keep, float scale, int sigmoid, int renorm,
-                         cudaStream_t stream) {
+                         int n_experts, int top, int groups, int keep, int group_top, float scale, int sigmoid, int renorm,
+                         float* gate_out, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
-    IDM_REQUIRE(n_experts > 0 && top > 0 && top <= n_experts && z_stride >= n_experts, "route: %d experts, %d per token, rows of %d",
-                n_experts, top, z_stride);
+    IDM_REQUIRE(n_experts > 0 && top > 0 && top <= n_experts && z_stride >= n_experts + (gate_out ? 1 : 0),
+                "route: %d experts, %d per token, rows of %d", n_experts, top, z_stride);
+    IDM_REQUIRE(group_top >= 1, "route: a group's score is the sum of its %d largest", group_top);
     IDM_REQUIRE(groups >= 1 && n_experts % groups == 0 && keep >= 1 && keep <= groups, "route: %d experts in %d groups of which %d are kept",
                 n_experts, groups, keep);
     const size_t smem = (size_t)RT_WARPS * (2 * n_experts + groups) * sizeof(float);
     IDM_REQUIRE(smem <= 160 * 1024, "route: %d experts do not fit shared memory", n_experts);
     if (smem > 48 * 1024) cudaFuncSetAttribute(route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     idm_launch(route_kernel, dim3((n_tokens + RT_WARPS - 1) / RT_WARPS), dim3(RT_WARPS * 32), smem, stream, z, z_stride, correction,
-               chosen, weight, n_tokens, n_experts, top, groups, keep, scale, sigmoid, renorm);
+               chosen, weight, n_tokens, n_experts, top, groups, keep, group_top, scale, sigmoid, renorm, gate_out);
     IDM_LAUNCH_CHECK("route");
     return 0;
 }

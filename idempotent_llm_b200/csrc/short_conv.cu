@@ -100,9 +100,13 @@ __global__ void __launch_bounds__(256) short_conv_kernel(ConvSeg g, ConvStep st,
 // 2 * half dims of every q and k head turned by the token's position (dim i with dim i + half; (u, v) ->
 // (u cos - v sin, v cos + u sin), table cs [N, half] of (cos, sin)), q stored [N, n_q, dk] and k, v written
 // to the token's place in the cache (pools [pages, n_kv, PAGE, dk] and [pages, n_kv, PAGE, dv]).
+// With `maps` > 1 a q or k head is that many parts side by side, each turned like a head of dk / maps dims, and q goes out as
+// one row per part, [N, n_q * maps, dk], zero outside its part: against the same key rows each such row scores its part
+// alone.
 struct ConvQkvArgs {
     ConvSeg seg; ConvStep st;
     int n_q, n_kv, dk, dv, half;
+    int maps;                       // parts of a q or k head that are turned each on its own (dk / maps dims each)
     const float2* cs;
     T* q_out; T* k_pool; T* v_pool;
     const int* table; int table_stride;
@@ -116,24 +120,33 @@ __global__ void __launch_bounds__(256) conv_qkv_cache_kernel(ConvQkvArgs a) {
     const ConvToken m = conv_token(a.st, t);                       // (one token per block: every thread the same)
     const size_t page = a.table[(size_t)m.slot * a.table_stride + m.pos / IDM_PAGE], prow = m.pos % IDM_PAGE;
     const int qk_heads = a.n_q + a.n_kv;
-    const int rest = a.dk - a.half;                       // work items of a q or k head: pairs, then single dims
+    const int part = a.dk / a.maps, per = part - a.half;  // work items of a part: pairs, then single dims
+    const int rest = a.maps * per;                        // work items of a q or k head
     const int qk_items = qk_heads * rest, v_items = a.n_kv * a.dv;
     // (steps of few tokens spread a token's items over several blocks: gridDim.y)
     for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < qk_items + v_items; i += gridDim.y * blockDim.x) {
         if (i < qk_items) {
-            const int head = i / rest, r = i % rest;
-            T* dst = head < a.n_q ? a.q_out + ((size_t)t * a.n_q + head) * a.dk
-                                  : a.k_pool + ((page * a.n_kv + (head - a.n_q)) * IDM_PAGE + prow) * (size_t)a.dk;
-            if (r < a.half) {
-                const float u = conv_at<TAPS>(a.seg, m, t, head * a.dk + r);
-                const float v = conv_at<TAPS>(a.seg, m, t, head * a.dk + r + a.half);
+            const int head = i / rest, mp = i % rest / per, r = i % per, d0 = mp * part;
+            const bool is_q = head < a.n_q;
+            T* row = is_q ? a.q_out + ((size_t)t * a.n_q + head) * a.maps * a.dk
+                          : a.k_pool + ((page * a.n_kv + (head - a.n_q)) * IDM_PAGE + prow) * (size_t)a.dk;
+            T* dst = row + (is_q ? mp * a.dk : 0) + d0;
+            const int other = r < a.half ? r + a.half : -1, d = r < a.half ? r : r + a.half;
+            if (other >= 0) {
+                const float u = conv_at<TAPS>(a.seg, m, t, head * a.dk + d0 + d);
+                const float v = conv_at<TAPS>(a.seg, m, t, head * a.dk + d0 + other);
                 const float2 cs = a.cs[(size_t)t * a.half + r];
-                from_f32(dst[r], u * cs.x - v * cs.y);
-                from_f32(dst[r + a.half], v * cs.x + u * cs.y);
+                from_f32(dst[d], u * cs.x - v * cs.y);
+                from_f32(dst[other], v * cs.x + u * cs.y);
             } else {
-                const int d = r + a.half;
-                from_f32(dst[d], conv_at<TAPS>(a.seg, m, t, head * a.dk + d));
+                from_f32(dst[d], conv_at<TAPS>(a.seg, m, t, head * a.dk + d0 + d));
             }
+            if (is_q)
+                for (int z = 0; z < a.maps; ++z)
+                    if (z != mp) {
+                        from_f32(row[z * a.dk + d0 + d], 0.f);
+                        if (other >= 0) from_f32(row[z * a.dk + d0 + other], 0.f);
+                    }
         } else {
             const int j = i - qk_items, g = j / a.dv, d = j % a.dv;
             T* dst = a.v_pool + ((page * a.n_kv + g) * IDM_PAGE + prow) * (size_t)a.dv;
@@ -199,7 +212,7 @@ extern "C" int idm_short_conv(const float* in, int in_stride, int col0, int chan
 }
 
 extern "C" int idm_conv_qkv_cache(const float* in, int in_stride, int col0, int taps, const float* w, float* state,
-                                  long long state_stride, int n_q, int n_kv, int dk, int dv, int half, const float* cs,
+                                  long long state_stride, int n_q, int n_kv, int dk, int dv, int half, int maps, const float* cs,
                                   void* q_out, void* k_pool, void* v_pool, const int* table, int table_stride,
                                   const int* token_seq, const int* positions, const int* slots, const int* q_start,
                                   const int* cu_q, int n_tokens, cudaStream_t stream) {
@@ -207,14 +220,14 @@ extern "C" int idm_conv_qkv_cache(const float* in, int in_stride, int col0, int 
     ConvQkvArgs a;
     const int channels = (n_q + n_kv) * dk + n_kv * dv;
     if (conv_seg(a.seg, "conv_qkv_cache", in, in_stride, col0, channels, taps, w, nullptr, state, state_stride)) return 1;
-    IDM_REQUIRE(n_q > 0 && n_kv > 0 && dk > 0 && dv > 0 && half >= 0 && 2 * half <= dk,
-                "conv_qkv_cache: heads %d/%d, sizes %d/%d, %d turning pairs", n_q, n_kv, dk, dv, half);
+    IDM_REQUIRE(n_q > 0 && n_kv > 0 && dk > 0 && dv > 0 && maps >= 1 && dk % maps == 0 && half >= 0 && 2 * half <= dk / maps,
+                "conv_qkv_cache: heads %d/%d, sizes %d/%d in %d parts, %d turning pairs", n_q, n_kv, dk, dv, maps, half);
     IDM_REQUIRE(half == 0 || cs != nullptr, "conv_qkv_cache: a rotation needs its table");
     a.st = ConvStep{token_seq, positions, slots, q_start, cu_q};
-    a.n_q = n_q; a.n_kv = n_kv; a.dk = dk; a.dv = dv; a.half = half; a.cs = (const float2*)cs;
+    a.n_q = n_q; a.n_kv = n_kv; a.dk = dk; a.dv = dv; a.half = half; a.maps = maps; a.cs = (const float2*)cs;
     a.q_out = (T*)q_out; a.k_pool = (T*)k_pool; a.v_pool = (T*)v_pool; a.table = table; a.table_stride = table_stride;
     // a block per token; with few tokens, several blocks per token, so that two blocks' worth of work per SM is about
-    const int items = (n_q + n_kv) * (dk - half) + n_kv * dv;
+    const int items = (n_q + n_kv) * (dk - maps * half) + n_kv * dv;
     int split = (296 + n_tokens - 1) / n_tokens;
     if (split > (items + 255) / 256) split = (items + 255) / 256;
     if (split < 1) split = 1;

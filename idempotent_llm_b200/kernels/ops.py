@@ -60,10 +60,10 @@ SIGNATURES = {
     "idm_embed": (c_int, "pppiip"),
     "idm_embed_scaled": (c_int, "ppppiifp"),
     "idm_post_pre_norm": (c_int, "pppfpfpiiip"),
-    "idm_gated_act": (c_int, "ppiiipp"),
+    "idm_gated_act": (c_int, "ppiiiffppp"),
     "idm_token_gate": (c_int, "pppiipiiip"),
     "idm_short_conv": (c_int, "piiiippipqppppppip"),
-    "idm_conv_qkv_cache": (c_int, "piiippqiiiiipppppipppppip"),
+    "idm_conv_qkv_cache": (c_int, "piiippqiiiiiipppppipppppip"),
     "idm_conv_state_update": (c_int, "piiiipqppppip"),
     "idm_ssd_chunk_tokens": (c_int, ""),
     "idm_ssd_scan": (c_int, "piiiipiiippppqpippiiiiippipip"),
@@ -79,6 +79,7 @@ SIGNATURES = {
     "idm_add_rmsnorm2": (c_int, "ppiqppfpppiip"),
     "idm_gemm_bf16_gated": (c_int, "pppiiiip"),
     "idm_gemm_bf16_gated_rows": (c_int, "pppiiiipp"),
+    "idm_gemm_bf16_gated_all": (c_int, "pppiiiiffppp"),
     "idm_add_rmsnorm": (c_int, "ppiqpfppiip"),
     "idm_rope_table": (c_int, "ppppiip"),
     "idm_qkv_finish": (c_int, "piqiiiippfpppppppiipppp"),
@@ -99,14 +100,18 @@ SIGNATURES = {
     "idm_attention_tc": (c_int, "ppppipippippppiiiifiiippiip"),
     "idm_attention_tc_sink": (c_int, "pppppipippippppiiiifiiippiip"),
     "idm_attention_tc_biased": (c_int, "ppppifiipppipippippppiiiifiiippiip"),
-    "idm_gate_scale": (c_int, "ppiifpiiiip"),
+    "idm_gate_scale": (c_int, "ppiifpiiiiiip"),
+    "idm_diff_combine": (c_int, "pfffpipiiiiip"),
+    "idm_retention_chunk_tokens": (c_int, ""),
+    "idm_retention_scratch_floats": (c_longlong, "iiii"),
+    "idm_retention": (c_int, "piiiipifppqpippiiiippipip"),
     "idm_attention_tc_status": (c_int, ""),
     "idm_attention_tc_set_few_rows": (c_int, "i"),
     "idm_latent_kv_finish": (c_int, "piiiiiipfpifppippppip"),
-    "idm_headwise": (c_int, "pqiipipiqiiiipifiip"),
+    "idm_headwise": (c_int, "pqiipipiqiiiipifpiiip"),
     "idm_latent_attention_max_rank": (c_int, ""),
     "idm_latent_attention_heads_per_block": (c_int, "iii"),
-    "idm_latent_attention": (c_int, "pppippppppiiiifiip"),
+    "idm_latent_attention": (c_int, "pppippppppiiiifiiip"),
     "idm_latent_expand_pack": (c_int, "pippiiiiiiipifippppipppip"),
     "idm_experts_few": (c_int, "pppppqqqpppiiiiiifip"),
     "idm_experts_major": (c_int, "pppppqqqppppiiiiiifip"),
@@ -117,7 +122,7 @@ SIGNATURES = {
     "idm_dense_ff": (c_int, "ppppppiiiip"),
     "idm_experts_combine": (c_int, "ppppiiifp"),
     "idm_rows_weight": (c_int, "pppip"),
-    "idm_route": (c_int, "pipppiiiiifiip"),
+    "idm_route": (c_int, "pipppiiiiiifiipp"),
     "idm_experts_identity": (c_int, "ppppiiiip"),
     "idm_post_layernorm": (c_int, "pppppfpiiip"),
     "idm_add_layernorm": (c_int, "ppiqppfppiip"),
@@ -272,17 +277,23 @@ class Kernels:
                                                hidden, self._stream()))
         return x
 
-    def gated_act(self, gu: torch.Tensor, act: int, row_w=None) -> torch.Tensor:
+    def _row_factors(self, n: int, *factors) -> None:
+        for f in factors:
+            if f is not None:
+                self._need(f, torch.float32, "row weights")
+                if f.numel() != n:
+                    raise KernelError(f"{f.numel()} row weights for {n} rows")
+
+    def gated_act(self, gu: torch.Tensor, act: int, row_w=None, row_out=None, limit: float = 0.0, slope: float = 0.0) -> torch.Tensor:
         """``act(gate) * up`` of a 32-bit gate/up product ``[N, 2 * inter]`` (gate columns, then up columns);
-        ``act``: 0 silu, 1 gelu (tanh form).  ``row_w [N]``: gate and up of a row are multiplied by it first."""
+        ``act``: 0 silu, 1 gelu (tanh form), 2 relu, 3 the clamped form with its constants ``limit`` and ``slope``.  ``row_w
+        [N]``: gate and up of a row are multiplied by it first; ``row_out [N]``: what the activation gives is."""
         self._need(gu, torch.float32, "gate-up")
         n, width = gu.shape
         y = torch.empty((n, width // 2), dtype=self.dtype, device=self.device)
-        if row_w is not None:
-            self._need(row_w, torch.float32, "row weights")
-            if row_w.numel() != n:
-                raise KernelError(f"{row_w.numel()} row weights for {n} rows")
-        self._check(self.lib.idm_gated_act(_p(gu), _p(y), n, width // 2, act, _p(row_w), self._stream()))
+        self._row_factors(n, row_w, row_out)
+        self._check(self.lib.idm_gated_act(_p(gu), _p(y), n, width // 2, act, float(limit), float(slope), _p(row_w), _p(row_out),
+                                           self._stream()))
         return y
 
     def token_gate(self, s, tokens, table, col0: int, act: int) -> torch.Tensor:
@@ -316,18 +327,19 @@ class Kernels:
                                             _p(ctx.slots), _p(ctx.q_start), _p(ctx.cu_q), n, self._stream()))
         return out
 
-    def conv_qkv_cache(self, proj, col0: int, w, state, n_q, n_kv, dk, dv, cs, kv, ctx) -> torch.Tensor:
+    def conv_qkv_cache(self, proj, col0: int, w, state, n_q, n_kv, dk, dv, cs, kv, ctx, maps: int = 1) -> torch.Tensor:
         """q, k, v channels of ``proj`` filtered, q and k turned by the rotary table ``cs [N, half, 2]`` (or None),
-        k and v written to the cache entry; returns q ``[N, n_q, dk]``."""
+        k and v written to the cache entry; returns q ``[N, n_q, dk]``.  ``maps``: a q or k head is that many parts side by
+        side, each turned on its own; q comes back as a row per part, zero outside it: ``[N, n_q * maps, dk]``."""
         self._need(proj, torch.float32, "projection")
         n, width = proj.shape
         half = 0 if cs is None else cs.shape[1]
         if cs is not None and (cs.shape[0] != n or cs.dtype != torch.float32):
             raise KernelError(f"rotary table {tuple(cs.shape)} does not match {n} tokens")
         self._check_kv(kv, n_kv, dk, dv)
-        q = torch.empty((n, n_q, dk), dtype=self.dtype, device=self.device)
+        q = torch.empty((n, n_q * maps, dk), dtype=self.dtype, device=self.device)
         self._check(self.lib.idm_conv_qkv_cache(_p(proj), width, col0, w.shape[1], _p(w), _p(state),
-                                                self._state_stride(state), n_q, n_kv, dk, dv, half, _p(cs), _p(q),
+                                                self._state_stride(state), n_q, n_kv, dk, dv, half, int(maps), _p(cs), _p(q),
                                                 _p(kv.k), _p(kv.v), _p(kv.table), kv.table.shape[1],
                                                 _p(ctx.token_seq), _p(ctx.positions), _p(ctx.slots), _p(ctx.q_start),
                                                 _p(ctx.cu_q), n, self._stream()))
@@ -346,9 +358,12 @@ class Kernels:
         [n_chunks + 1], each sequence's first chunk [n_seqs + 1], n_chunks), on the device, made once a step; None
         when no sequence brings more than a chunk's tokens (then every sequence runs token by token from its state)."""
         L = self.lib.idm_ssd_chunk_tokens()
-        if ctx.single_token or ctx.max_q_len <= L:
-            return None
-        plan = ctx.memo.get("ssd_chunks")
+        return None if ctx.single_token or ctx.max_q_len <= L else self._chunks(ctx, L)
+
+    def _chunks(self, ctx, L: int):
+        """Portions cut into chunks of ``L`` tokens: what ``ssd_chunks`` returns."""
+        key = ("chunks", L)
+        plan = ctx.memo.get(key)
         if plan is None:
             borders, first, at = [], [0], 0
             for n in ctx.host_q_lens:
@@ -357,7 +372,7 @@ class Kernels:
                 first.append(len(borders))
             borders.append(at)
             dev = torch.tensor(borders + first, dtype=torch.int32).to(self.device)
-            plan = ctx.memo["ssd_chunks"] = (dev, dev[:len(borders)], dev[len(borders):], len(borders) - 1)
+            plan = ctx.memo[key] = (dev, dev[:len(borders)], dev[len(borders):], len(borders) - 1)
         return plan
 
     def ssd_scan(self, xbc, cols, proj, z_col: int, dt_col: int, dt_bias, a_log, d_skip, state, ctx, heads, groups,
@@ -381,6 +396,44 @@ class Kernels:
                                           ctx.n_seqs, heads, groups, P, N, _p(chunk_t0), _p(seq_chunk0), n_chunks,
                                           _p(scratch), n, self._stream()), 3 if n_chunks else 1)
         return y
+
+    # portions of up to so many tokens are walked token by token, longer ones run in chunks side by side
+    RETENTION_WALK = 8
+
+    def retention(self, proj, cols, cs, k_scale: float, decay, state, ctx, H: int, dk: int, dv: int) -> torch.Tensor:
+        """``S <- decay S + k v^T; o = S^T q`` per head over the step's tokens, from and to each sequence's state ``[slots, H *
+        dk * dv]``: q, k, v at columns ``cols`` of the 32-bit ``proj``, q and k turned by the table ``cs [N, half, 2]`` (or None), k
+        times ``k_scale``; returns ``o [N, H * dv]`` in 32-bit.  Steps with long portions run them in chunks side by side, and
+        turn q and k in ``proj`` in place."""
+        self._need(proj, torch.float32, "projection")
+        self._need(decay, torch.float32, "decays")
+        n, width = proj.shape
+        half = 0 if cs is None else cs.shape[1]
+        if decay.numel() != H or (cs is not None and (cs.dtype != torch.float32 or tuple(cs.shape) != (n, half, 2))):
+            raise KernelError(f"retention: {decay.numel()} decays for {H} heads, a table of {None if cs is None else tuple(cs.shape)}")
+        o = torch.empty((n, H * dv), dtype=torch.float32, device=self.device)
+        chunk_t0 = seq_chunk0 = scratch = None
+        n_chunks = 0
+        if not ctx.single_token and ctx.max_q_len > self.RETENTION_WALK:
+            _, chunk_t0, seq_chunk0, n_chunks = self._chunks(ctx, self.lib.idm_retention_chunk_tokens())
+            scratch = self.scratch("retention", int(self.lib.idm_retention_scratch_floats(n_chunks, H, dk, dv)))
+        self._check(self.lib.idm_retention(_p(proj), width, *cols, _p(cs), half, float(k_scale), _p(decay), _p(state),
+                                           self._state_stride(state), _p(o), H * dv, _p(ctx.cu_q), _p(ctx.slots), ctx.n_seqs, H,
+                                           dk, dv, _p(chunk_t0), _p(seq_chunk0), n_chunks, _p(scratch), n, self._stream()),
+                    4 if n_chunks else 1)
+        return o
+
+    def diff_combine(self, o, lam: float, eps: float, post: float, gate, gate_stride: int, out, out_col: int, H: int, dv: int) -> None:
+        """Two contexts per head (``o [N, 2 * H * dv]``, head by head) into one: ``a1 - lam a2`` over its root mean square, times
+        ``post`` and the sigmoid of the head's gate (a 32-bit view with row stride ``gate_stride``, or None), into columns
+        ``out_col ..`` of ``out``."""
+        self._need(o, self.dtype, "the maps' contexts")
+        self._need(out, self.dtype, "mixer output")
+        n, width = o.shape
+        if width != 2 * H * dv:
+            raise KernelError(f"diff_combine: rows of {width} for {H} heads of two maps of {dv}")
+        self._check(self.lib.idm_diff_combine(_p(o), float(lam), float(eps), float(post), (gate.data_ptr() if gate is not None else None),
+                                              gate_stride, _p(out), out.shape[1], out_col, n, H, dv, self._stream()))
 
     def ssd_group_norm(self, y, parts: int, w, eps: float, scale: float, out, out_col: int) -> None:
         """``out[:, out_col : out_col + width] = rmsnorm over each of `parts` equal parts of y * w * scale``."""
@@ -488,7 +541,7 @@ class Kernels:
     def delta_out(self, o, w, eps: float, gate, gate_col: int, scale: float, out, out_col: int, H: int, dv: int,
                   gate_act: int = 0) -> None:
         """``out[:, out_col ..] = rmsnorm over each head of o * w * act(gate columns) * scale``; ``gate_act`` 0: sigmoid,
-        1: silu."""
+        1: silu; ``w`` None: ones."""
         n = o.shape[0]
         self._check(self.lib.idm_delta_out(_p(o), o.shape[1], _p(w), float(eps), _p(gate), gate.shape[1], gate_col,
                                            int(gate_act), float(scale), _p(out), out.shape[1], out_col, n, H, dv, self._stream()))
@@ -511,14 +564,17 @@ class Kernels:
                                               _p(x2), _p(post), n, hidden, self._stream()))
         return x1, x2
 
-    def gemm_gated(self, x, w_tiled, inter: int, act: int) -> torch.Tensor:
-        """``act(x . gate^T) * (x . up^T)`` in the storage dtype ``[M, inter]`` (``tile_gate_up`` layout)."""
+    def gemm_gated(self, x, w_tiled, inter: int, act: int, row_out=None, limit: float = 0.0, slope: float = 0.0) -> torch.Tensor:
+        """``act(x . gate^T) * (x . up^T)`` in the storage dtype ``[M, inter]`` (``tile_gate_up`` layout); ``row_out``, ``limit``,
+        ``slope`` as in ``gated_act``."""
         M, N, Kd = self._gemm_shape(x, w_tiled)
         if N != -(-inter // 64) * 128:
             raise KernelError(f"tiled gate/up weight has {N} rows, expected {-(-inter // 64) * 128}")
         y = torch.empty((M, inter), dtype=self.dtype, device=self.device)
+        self._row_factors(M, row_out)
         if M:
-            self._check(self.lib.idm_gemm_bf16_gated(_p(x), _p(w_tiled), _p(y), M, inter, Kd, act, self._stream()))
+            self._check(self.lib.idm_gemm_bf16_gated_all(_p(x), _p(w_tiled), _p(y), M, inter, Kd, act, float(limit), float(slope),
+                                                         None, _p(row_out), self._stream()))
         return y
 
     def add_rmsnorm(self, h, delta, gamma, eps: float, rows=None) -> torch.Tensor:
@@ -660,15 +716,18 @@ class Kernels:
         return (self.dtype == torch.bfloat16 and self.attention_impl == "tcgen05" and hd == dv and kv.ring == 0
                 and bool(self.lib.idm_attention_tc_supports(hd)))
 
-    def gate_scale(self, o, gate, gate_stride: int, scale: float, out, out_col: int, gate_group: int = 1) -> None:
+    def gate_scale(self, o, gate, gate_stride: int, scale: float, out, out_col: int, gate_group: int = 1, in_head: int = 1,
+                   out_head: int = 1) -> None:
         """``out[:, out_col : out_col + width] = o * sigmoid(gate) * scale`` (``gate``: a 32-bit view with row stride
         ``gate_stride``, or None for the constant alone; ``gate_group`` columns in a row share one gate number: a head's
-        size for a gate per head)."""
+        size for a gate per head).  ``in_head`` / ``out_head``: heads of ``in_head`` elements in ``o`` of which the first ``out_head``
+        count; ``out`` and ``gate`` hold those alone."""
         self._need(o, self.dtype, "mixer output")
         self._need(out, self.dtype, "gated output")
         n, width = o.shape
+        width = width // in_head * out_head
         self._check(self.lib.idm_gate_scale(_p(o), (gate.data_ptr() if gate is not None else None), gate_stride, int(gate_group),
-                                            float(scale), _p(out), out.shape[1], out_col, n, width, self._stream()))
+                                            float(scale), _p(out), out.shape[1], out_col, n, width, int(in_head), int(out_head), self._stream()))
 
     def attention_tc_plan(self, ctx, n_q: int, n_kv: int, hd: int, through_scratch=None, share=None, chunk=None):
         """What the attention launches of one step share, for one arrangement of heads: the list of tiles
@@ -1022,10 +1081,11 @@ class Kernels:
         return rows
 
     def headwise(self, x, x_col: int, n_heads: int, head_stride: int, w, tail: int = 0, rot_dims: int = 0, cs=None,
-                 mag: float = 1.0, out_f32: bool = False, halves: bool = False) -> torch.Tensor:
+                 mag: float = 1.0, out_f32: bool = False, halves: bool = False, gate=None, gate_stride: int = 0) -> torch.Tensor:
         """A matrix per head: ``out[t, h, :O] = x[t, x_col + h * head_stride : ... + I] . w[h]`` with ``w [H, I, O]``;
         ``tail`` more columns of ``x`` behind a head's ``I`` are copied behind its outputs, the first ``rot_dims`` of them
-        turned.  ``x`` 32-bit ``[N, ld]``; returns ``[N, H, O + tail]`` (32-bit or the storage dtype)."""
+        turned.  ``x`` 32-bit ``[N, ld]``; returns ``[N, H, O + tail]`` (32-bit or the storage dtype).  ``gate``: a 32-bit view ``[N, H *
+        O]`` with row stride ``gate_stride`` whose sigmoids multiply the outputs."""
         self._need(x, torch.float32, "headwise input")
         self._need(w, self.dtype, "headwise matrices")
         n, ld = x.shape
@@ -1035,14 +1095,15 @@ class Kernels:
         out = torch.empty((n, H, O + tail), dtype=torch.float32 if out_f32 else self.dtype, device=self.device)
         half = 0 if cs is None else cs.shape[1]
         self._check(self.lib.idm_headwise(x.data_ptr() + 4 * x_col, ld, head_stride, I, _p(w), O, _p(out), 1 if out_f32 else 0,
-                                          H * (O + tail), O + tail, tail, rot_dims, 1 if halves else 0, _p(cs), half, float(mag), n, H,
-                                          self._stream()))
+                                          H * (O + tail), O + tail, tail, rot_dims, 1 if halves else 0, _p(cs), half, float(mag),
+                                          (gate.data_ptr() if gate is not None else None), int(gate_stride), n, H, self._stream()))
         return out
 
-    def latent_attention(self, qa, kv, ctx, rank: int, scale: float, sink=None) -> torch.Tensor:
+    def latent_attention(self, qa, kv, ctx, rank: int, scale: float, sink=None, window=None) -> torch.Tensor:
         """Causal attention of the step's queries ``qa [N, H, D]`` (32-bit, in the latent's space) over the cached rows
         ``[c | r]`` of ``D`` numbers; returns the context ``[N, H * rank]`` in 32-bit: the weighted sums of ``c``.
-        Steps of few tokens cut the keys into runs of 64 to 256 positions, a block each, that meet in scratch."""
+        Steps of few tokens cut the keys into runs of 64 to 256 positions, a block each, that meet in scratch.  ``window``: a
+        query sees itself and the ``window - 1`` rows before it."""
         self._need(qa, torch.float32, "latent queries")
         n, H, D = qa.shape
         if tuple(kv.k.shape[1:]) != (1, self.page, D):
@@ -1057,17 +1118,21 @@ class Kernels:
         if groups < 2 * self.sm_count:
             # runs short enough to give the step about four blocks per SM, of 64 to 256 keys (whole pages); the
             # choice depends on the step's shape and the cache's limit only, never on a sequence's length
-            fair = -(-ctx.max_kv_len * groups // (4 * self.sm_count))
+            longest = min(ctx.max_kv_len, int(window)) if window else ctx.max_kv_len
+            fair = -(-longest * groups // (4 * self.sm_count))
             run_keys = min(256, max(64, -(-fair // 64) * 64))
-            run_keys = max(run_keys, -(-ctx.max_kv_len // (512 * 64)) * 64)       # (at most 512 runs)
+            run_keys = max(run_keys, -(-longest // (511 * 64)) * 64)              # (at most 512 runs)
             n_runs = max(1, -(-ctx.max_kv_len // run_keys))
+            if window:                                                            # (a window starts anywhere in its first run)
+                n_runs = min(n_runs, (longest + run_keys - 2) // run_keys + 1)
         if n_runs > 1:
             part = self.scratch("latent_attention", n * H * n_runs * (rank + 2))
         else:
             run_keys = 1 << 30
         self._check(self.lib.idm_latent_attention(_p(qa), _p(kv.k), _p(kv.table), kv.table.shape[1], _p(ctx.token_seq),
                                                   _p(ctx.positions), _p(ctx.slots), _p(sink), _p(out), _p(part), n, H, rank,
-                                                  D, scale, run_keys, n_runs, self._stream()), 2 if n_runs > 1 else 1)
+                                                  D, scale, run_keys, n_runs, int(window) if window else 0, self._stream()),
+                    2 if n_runs > 1 else 1)
         return out
 
     def latent_expand_pack(self, proj, up, rows, H, dn, dr, dv, R, rot_dims, cs, mag, hd, table, n_pages, ctx, halves: bool = False):
@@ -1188,21 +1253,30 @@ class Kernels:
         n, width = h.shape
         self._check(self.lib.idm_experts_combine(_p(z), _p(place), _p(pair_w), _p(h), n, width, place.shape[1], float(weight), self._stream()))
 
-    def route(self, z, correction, top: int, groups: int, keep: int, scale: float, sigmoid: bool = False, renorm: bool = True):
+    def route(self, z, correction, top: int, groups: int, keep: int, scale: float, sigmoid: bool = False, renorm: bool = True,
+              group_top: int = 1, n_experts: Optional[int] = None):
         """From 32-bit router logits ``z [N, E]`` to the experts each token uses: softmax over all E, choice by
         ``softmax + correction`` among the experts of the ``keep`` best of ``groups`` equal groups of neighbours, the
         ``top`` best in descending order; returns ``(chosen [N, top] int32, weight [N, top])`` with the weights the
         chosen experts' softmax values over their sum, times ``scale``.  ``sigmoid``: element by element instead of the
-        softmax; ``renorm`` False: the chosen values times ``scale`` as they are."""
+        softmax; ``renorm`` False: the chosen values times ``scale`` as they are.  ``group_top``: a group's score is the sum of
+        its so many largest choice scores.  ``n_experts`` one less than the logits' columns: the last column is a gate, and its
+        sigmoids ``[N]`` are returned as a third result."""
         self._need(z, torch.float32, "router logits")
         n, E = z.shape
+        gate = None
+        if n_experts is not None and n_experts != E:
+            if n_experts != E - 1:
+                raise KernelError(f"route: {E} columns for {n_experts} experts and a gate")
+            E, gate = n_experts, torch.empty((n,), dtype=torch.float32, device=self.device)
         if correction is not None and (correction.dtype != torch.float32 or correction.numel() != E):
             raise KernelError(f"route: the correction must hold one 32-bit number for each of the {E} experts")
         chosen = torch.empty((n, top), dtype=torch.int32, device=self.device)
         weight = torch.empty((n, top), dtype=torch.float32, device=self.device)
         self._check(self.lib.idm_route(_p(z), z.stride(0), _p(correction), _p(chosen), _p(weight), n, E, int(top), int(groups),
-                                       int(keep), float(scale), 1 if sigmoid else 0, 1 if renorm else 0, self._stream()))
-        return chosen, weight
+                                       int(keep), int(group_top), float(scale), 1 if sigmoid else 0, 1 if renorm else 0, _p(gate),
+                                       self._stream()))
+        return (chosen, weight) if gate is None else (chosen, weight, gate)
 
     def experts_identity(self, x, chosen, weight, h, n_real: int) -> None:
         """``h[t] += x[t] * (the weights of t's pairs whose expert number is at least n_real)``: experts that hand

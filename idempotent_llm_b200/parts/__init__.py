@@ -9,6 +9,8 @@ from .mlp import DenseMLP, GatedMLP
 from .block import PreNormBlock
 from .sink_attention import SinkAttention
 from .ssd import SSDMixer
+from .retention import Retention
+from .differential_attention import DifferentialAttention
 from .parallel import ParallelMixer
 from .sandwich import SandwichBlock, TokenSide
 from .latent_attention import LatentAttention
@@ -25,4 +27,4 @@ __all__ = ["BLOCKS", "FEED_FORWARDS", "MIXERS", "NORMS", "POSITIONS", "Block", "
            "GatedMLP", "PreNormBlock", "SinkAttention", "SSDMixer", "ParallelMixer", "SandwichBlock", "TokenSide",
            "DyT", "DenseMLP", "LatentAttention", "TableExperts", "HeadAttention", "GatedDeltaRule",
            "ParallelResidualBlock", "EMBEDDINGS", "CastStream", "LayerNorm", "RoutedExperts", "BigramHashEmbedding",
-           "PostNormBlock", "GroupedRMSNorm", "SumNormBlock"]
+           "PostNormBlock", "GroupedRMSNorm", "SumNormBlock", "Retention", "DifferentialAttention"]

@@ -138,13 +138,15 @@ class RoutedExperts(FeedForward):
     captured single-token step needs nothing from the host.  The experts then run the way table-routed experts do, on
     the same kernels: a step's row numbers take the place of token ids and the step's choices the place of the table;
     every (token, choice) pair carries its weight.  Steps of many tokens, outside a captured graph, read the choices
-    back and group the rows by expert for one matrix product per expert.  Returns the sum as a delta (a norm may sit
-    behind the feed-forward).
+    back and group the rows by expert for one matrix product per expert.  The sum goes into the stream, or is returned as
+    a delta where a norm sits behind the feed-forward.
 
     Options: ``s = sigmoid(z)`` instead of the softmax, no correction, weights left as they are (not over their sum), and
     the weight on an expert's input, ``expert(w_k x_t)``: gate and up are linear, so w_k multiplies both of the pair's
-    pre-activations in 32-bit, in the epilogue of the product that makes them."""
+    pre-activations in 32-bit, in the epilogue of the product that makes them.  A gate on the shared expert (one number per
+    token) is one more row of the router's matrix; its sigmoid multiplies what the shared expert's activation gives."""
 
+    accepts_residual = True
     same_bits_across_steps = False      # whole prompts, portions and single tokens take different kernels
 
     @classmethod
@@ -160,6 +162,8 @@ class RoutedExperts(FeedForward):
                   TensorDecl(p + nm.down, (s.hidden, s.intermediate))]
         if s.shared is not None:
             d += FEED_FORWARDS.get(s.shared.kind).declare(s.shared, prefix)
+            if s.shared_gate is not None:
+                d.append(TensorDecl(prefix + s.shared_gate, (1, s.hidden)))
         return d
 
     def __init__(self, spec, weights, prefix, rt):
@@ -173,6 +177,8 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"routed experts: {s.top} experts cannot come from {s.groups_keep} groups of {total // s.groups}")
         if s.scores not in ("softmax", "sigmoid") or s.weight_on not in ("output", "input"):
             raise ValueError(f"routed experts: scores={s.scores!r}, weight_on={s.weight_on!r} are not built")
+        if s.group_top < 1 or (s.shared_gate is not None and s.shared is None):
+            raise ValueError(f"routed experts: group_top={s.group_top}, a gate {s.shared_gate!r} on the shared expert {s.shared}")
         if s.weight_on == "input" and s.n_identity:
             raise ValueError("routed experts: a weight on the input and identity experts do not come together")
         self.weight_in = s.weight_on == "input"
@@ -194,6 +200,8 @@ class RoutedExperts(FeedForward):
                 self.row_stride, self.up_off = s.hidden, s.intermediate * s.hidden
             self.down = torch.stack(stack(nm.down)).contiguous()
         self.w_router = weights[prefix + s.router].to(rt.dtype).contiguous()
+        if s.shared_gate is not None:
+            self.w_router = torch.cat([self.w_router, weights[prefix + s.shared_gate].to(rt.dtype)], dim=0).contiguous()
         self.correction = None if s.correction is None else weights[prefix + s.correction].to(torch.float32).contiguous()
         self.shared = None
         if s.shared is not None:
@@ -208,21 +216,29 @@ class RoutedExperts(FeedForward):
         return r
 
     def route(self, x):
-        """(chosen [N, top] int32, weight [N, top]) of the step's rows."""
+        """(chosen [N, top] int32, weight [N, top]) of the step's rows, and with a gated shared expert its gates [N]."""
         s, K = self.spec, self.rt.kernels
-        z = K.gemm_store(x, self.w_router, pad=True)                        # 32-bit logits over all experts
+        z = K.gemm_store(x, self.w_router, pad=True)                        # 32-bit logits over all experts (and the gate's)
         return K.route(z, self.correction, s.top, s.groups, s.groups_keep, s.scale, sigmoid=s.scores == "sigmoid",
-                       renorm=s.renormalize)
+                       renorm=s.renormalize, group_top=s.group_top, n_experts=s.n_experts + s.n_identity)
 
-    def forward(self, x, ctx):
+    def forward(self, x, ctx, residual=None):
+        """Adds into ``residual`` and returns None, or returns the sum as a delta ``[1, N, hidden]``."""
         s, K = self.spec, self.rt.kernels
         n = x.shape[0]
-        # the shared expert's output opens the sum (its product writes the buffer the experts then add into)
+        chosen, weight, *gate = self.route(x)
+        # the shared expert's output opens the sum: its product writes the buffer the experts then add into (or adds into
+        # the stream, where the experts' kernels add as well)
+        h = residual
         if self.shared is not None:
-            h = self.shared.forward(x, ctx)[0]
-        else:
+            d = self.shared.forward(x, ctx, residual=residual, **({"row_out": gate[0]} if gate else {}))
+            if d is not None:
+                if residual is None:
+                    h = d[0]
+                else:
+                    residual += d[0]
+        elif residual is None:
             h = torch.zeros((n, s.hidden), dtype=torch.float32, device=x.device)
-        chosen, weight = self.route(x)
         if s.n_experts:
             rows = self._row_numbers(n, x.device)
             in_eager_step = getattr(ctx, "host_tokens", None) is not None
@@ -235,7 +251,7 @@ class RoutedExperts(FeedForward):
                               pair_w=weight, weight_in=self.weight_in)
         if s.n_identity:
             K.experts_identity(x, chosen, weight, h, s.n_experts)
-        return h.unsqueeze(0)
+        return None if residual is not None else h.unsqueeze(0)
 
     def _grouped(self, x, chosen, weight, h):
         s, K = self.spec, self.rt.kernels

@@ -7,9 +7,10 @@ In this file's notation, for the mixer's input h of one sequence (positions t = 
     c_t             = a_t / sqrt(mean(a_t^2) + eps) * g
     r_t             = turn(b_t, t),  qr <- turn(qr, t)        pairs j by angle t f_j, times a magnitude: neighbours (2j, 2j+1),
                                                               or dims (j, j + dims / 2)
-    s_tj            = scale * (qn_i . Uk_i c_j + qr_i . r_j)   (j <= t)
+    s_tj            = scale * (qn_i . Uk_i c_j + qr_i . r_j)   (t - window < j <= t)
     w_tj            = exp(s_tj) / (sum_j' exp(s_tj') [+ exp(sink_i)])
-    out_t           = Wo [.. | Uv_i sum_j w_tj c_j | ..]
+    o_t             = [.. | Uv_i sum_j w_tj c_j | ..] [* sigmoid(Wg h_t)]
+    out_t           = Wo o_t
 
 A token keeps the row ``[c_t | r_t]`` and nothing per head.  The kernels work in the latent's space: the query
 becomes ``[Uk_i^T qn_i | qr_i]``, every head scores the same cached rows, the context is a weighted sum of ``c``, and
@@ -47,6 +48,8 @@ class LatentAttention(Mixer):
              TensorDecl(prefix + nm.up_v, (s.n_heads * s.value_dim, s.kv_rank))]
         if s.sink:
             d.append(TensorDecl(prefix + nm.sink, (s.n_heads,), init="unit_normal"))
+        if s.gate:
+            d.append(TensorDecl(prefix + nm.gate, (s.n_heads * s.value_dim, s.hidden)))
         d.append(TensorDecl(prefix + nm.o, (s.hidden, s.n_heads * s.value_dim)))
         return d
 
@@ -74,9 +77,11 @@ class LatentAttention(Mixer):
             self.rot_dims = s.position.dim
             self.magnitude = float(getattr(self.position, "magnitude", 1.0))
         H, dn, dv, R = s.n_heads, s.plain_dim, s.value_dim, s.kv_rank
-        # q and the down projection are one product (rows one after another)
-        self.w_in = torch.cat([weights[prefix + nm.q].to(rt.dtype), weights[prefix + nm.down].to(rt.dtype)], dim=0).contiguous()
+        # q, the down projection and the gate are one product (rows one after another)
+        mats = [weights[prefix + n].to(rt.dtype) for n in (nm.q, nm.down) + ((nm.gate,) if s.gate else ())]
+        self.w_in = torch.cat(mats, dim=0).contiguous()
         self.q_cols = H * (dn + s.rot_dim)
+        self.gate_col = self.q_cols + R + s.rot_dim
         self.down_norm = weights[prefix + nm.down_norm].to(torch.float32).contiguous()
         # per head [in, out] with `out` contiguous: Uk_i as stored (plain_dim x rank), Uv_i transposed (rank x value_dim)
         self.uk = weights[prefix + nm.up_k].to(rt.dtype).reshape(H, dn, R).contiguous()
@@ -127,11 +132,16 @@ class LatentAttention(Mixer):
         q, k, v = K.latent_expand_pack(proj, up, rows, s.n_heads, s.plain_dim, s.rot_dim, s.value_dim, s.kv_rank,
                                        self.rot_dims, cs, self.magnitude, hd, table, n_pages, ctx, halves=self.halves)
         own = KVView(k=k, v=v, table=table, ring=0, n_kv_heads=s.n_heads, head_dim=hd, window=None)
-        o = K.attention_tc(q, own, ctx, s.softmax_scale, sink=self.sink)    # [N, H * hd]
+        o = K.attention_tc(q, own, ctx, s.softmax_scale, sink=self.sink, window=s.window)    # [N, H * hd]
+        w_o = self.w_o_padded
+        if s.gate:                      # the gate's pass also drops the heads' padding
+            g = torch.empty((o.shape[0], s.n_heads * s.value_dim), dtype=self.rt.dtype, device=o.device)
+            K.gate_scale(o, proj[:, self.gate_col:], proj.shape[1], 1.0, g, 0, in_head=hd, out_head=s.value_dim)
+            o, w_o = g, self.w_o
         if residual is not None:
-            K.gemm_residual(o, self.w_o_padded, residual)
+            K.gemm_residual(o, w_o, residual)
             return None
-        return K.gemm(o, self.w_o_padded)
+        return K.gemm(o, w_o)
 
     def forward(self, x, ctx, kv, state, writes_cache: bool, residual=None):
         """Returns the delta ``[1, N, hidden]``, or None after adding it into ``residual`` in place."""
@@ -147,8 +157,9 @@ class LatentAttention(Mixer):
         # queries into the latent's space, their rotated part turned: [N, H, rank + rot_dim], 32-bit
         qa = K.headwise(proj, 0, s.n_heads, s.plain_dim + s.rot_dim, self.uk, tail=s.rot_dim, rot_dims=self.rot_dims,
                         cs=cs, mag=self.magnitude, out_f32=True, halves=self.halves)
-        c = K.latent_attention(qa, kv, ctx, s.kv_rank, s.softmax_scale, sink=self.sink)     # 32-bit [N, H * rank]
-        o = K.headwise(c, 0, s.n_heads, s.kv_rank, self.uv_t).view(x.shape[0], s.n_heads * s.value_dim)
+        c = K.latent_attention(qa, kv, ctx, s.kv_rank, s.softmax_scale, sink=self.sink, window=s.window)     # 32-bit [N, H * rank]
+        gate = {"gate": proj[:, self.gate_col:], "gate_stride": proj.shape[1]} if s.gate else {}
+        o = K.headwise(c, 0, s.n_heads, s.kv_rank, self.uv_t, **gate).view(x.shape[0], s.n_heads * s.value_dim)
         if residual is not None and getattr(K, "fused", False) and not self.pad:
             K.gemm_residual(o, self.w_o, residual)
             return None

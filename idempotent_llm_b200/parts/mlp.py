@@ -13,6 +13,7 @@ from .base import FEED_FORWARDS, FeedForward
 
 # the kernels' numbers of the gated activations (csrc/common.cuh: gated_act)
 ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu": 2}
+CLAMPED = 3             # "clamped": both branches bounded, with constants of its own (a dense feed-forward's only)
 
 
 @FEED_FORWARDS.register("gated_mlp")
@@ -27,9 +28,12 @@ class GatedMLP(FeedForward):
                 TensorDecl(prefix + nm.down, (spec.hidden, spec.intermediate))]
 
     def __init__(self, spec, weights, prefix, rt):
-        if spec.activation not in ACTIVATIONS:
-            raise ValueError(f"activation {spec.activation!r} is not built; known: {sorted(ACTIVATIONS)}")
-        self.act = ACTIVATIONS[spec.activation]
+        if spec.activation not in ACTIVATIONS and spec.activation != "clamped":
+            raise ValueError(f"activation {spec.activation!r} is not built; known: {sorted(ACTIVATIONS) + ['clamped']}")
+        self.act = CLAMPED if spec.activation == "clamped" else ACTIVATIONS[spec.activation]
+        self.consts = {"limit": spec.limit, "slope": spec.slope} if self.act == CLAMPED else {}
+        if self.act == CLAMPED and not spec.limit >= 0:
+            raise ValueError(f"a clamped activation's limit must not be negative, got {spec.limit}")
         self.spec = spec
         self.rt = rt
         nm = spec.names
@@ -57,18 +61,21 @@ class GatedMLP(FeedForward):
         prog.gemm_swiglu(x, self.w_gate_up, s.hidden, s.intermediate, y)
         prog.gemm_residual(y, self.w_down, s.intermediate, h)
 
-    def forward(self, x, ctx, residual=None):
-        """Returns the delta ``[P, N, hidden]``, or None after adding it into ``residual`` in place."""
+    def forward(self, x, ctx, residual=None, row_out=None):
+        """Returns the delta ``[P, N, hidden]``, or None after adding it into ``residual`` in place.  ``row_out [N]``: a 32-bit
+        factor per token on the result (the down projection is linear, so it multiplies that projection's input, where the
+        activation is made)."""
         K = self.rt.kernels
         if self.fused:
-            y = (K.gemm_swiglu(x, self.w_gate_up, self.spec.intermediate) if self.act == 0
-                 else K.gemm_gated(x, self.w_gate_up, self.spec.intermediate, self.act))
+            y = (K.gemm_swiglu(x, self.w_gate_up, self.spec.intermediate) if self.act == 0 and row_out is None
+                 else K.gemm_gated(x, self.w_gate_up, self.spec.intermediate, self.act, row_out=row_out, **self.consts))
             if residual is not None:
                 K.gemm_residual(y, self.w_down, residual)
                 return None
             return K.gemm(y, self.w_down)
         gu = K.gemm(x, self.w_gate_up, **self.pad)          # [P, N, 2 * intermediate]
-        y = K.swiglu(gu) if self.act == 0 else K.gated_act(gu[0], self.act)      # [N, intermediate]
+        y = (K.swiglu(gu) if self.act == 0 and row_out is None
+             else K.gated_act(gu[0], self.act, row_out=row_out, **self.consts))     # [N, intermediate]
         return K.gemm(y, self.w_down, **self.pad)           # [P, N, hidden]
 
 

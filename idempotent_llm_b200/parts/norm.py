@@ -21,12 +21,14 @@ from .base import NORMS, CastStream, Norm, NormedDelta
 class RMSNorm(Norm):
     @classmethod
     def declare(cls, spec, prefix):
-        return [TensorDecl(prefix + spec.weight, (spec.size,), init="one_plus_normal")]
+        return [TensorDecl(prefix + spec.weight, (spec.size,), init="normal" if spec.weight_offset else "one_plus_normal")]
 
     def __init__(self, spec, weights, prefix, rt):
         self.spec = spec
         self.rt = rt
         self.weight = weights[prefix + spec.weight].to(torch.float32).contiguous()
+        if spec.weight_offset:                    # the tensor is an offset from a constant: the sum once, in 32-bit
+            self.weight = self.weight + float(spec.weight_offset)
 
     def forward(self, h, delta, ctx, rows=None):
         if isinstance(delta, CastStream):

@@ -83,6 +83,8 @@ def _register_builtin() -> None:
     register_architecture(PUNUNEX, PununexConfig)
     from .config.tosodra import ARCHITECTURE as TOSODRA, TosodraConfig
     register_architecture(TOSODRA, TosodraConfig)
+    from .config.zazulix import ARCHITECTURE as ZAZULIX, ZazulixConfig
+    register_architecture(ZAZULIX, ZazulixConfig)
 
 
 _register_builtin()
