@@ -183,7 +183,7 @@ def decode_point(lm, lens, steps: int, warmup: int, seed: int, repeats: int = 1,
     ms = statistics.median(times)
     sess.finish()
     mean_len = sum(l + warmup + repeats * steps / 2 for l in lens)
-    kv_read = (cache_bytes_read(lm, [l + warmup + repeats * steps / 2 for l in lens]) if getattr(cfg, "architecture", "") in ("Fuginex", "Tosodra")
+    kv_read = (cache_bytes_read(lm, [l + warmup + repeats * steps / 2 for l in lens]) if getattr(cfg, "architecture", "") in ("Fuginex", "Tosodra", "Zazulix")
                else kv_bytes_per_token(eng) * mean_len)
     bytes_step = step_weight_bytes(lm, batch) + kv_read + 2 * batch * state_bytes_per_sequence(eng)
     toks = sess.tokens()
@@ -333,6 +333,37 @@ def tosodra_prefill_flops(cfg, lens) -> float:
     return total + 2 * W * cfg.vocab * len(lens)
 
 
+def zazulix_prefill_flops(cfg, lens) -> float:
+    """The same count for a Zazulix configuration, per layer: the mixer's input and output projections (with the gate); for
+    a latent layer every head's keys and values from the latent and attention over the window; for a differential one two
+    maps over all earlier keys; for a retention the recurrence (per token, head, key channel and value column: decay, write
+    and read-out); the dense feed-forward, or the router, `top` experts and the shared expert."""
+    W, tokens, total = cfg.width, sum(lens), 0.0
+
+    def seen(t, window):
+        if window is None or window >= t:
+            return t * (t + 1) // 2
+        return window * (window + 1) // 2 + (t - window) * window
+    for L in cfg.layers:
+        f, linear = L.mlp, 0
+        if f is not None:
+            linear += 3 * W * f.ff if f.kind == "dense" else W * f.experts + 3 * W * f.ff * f.top + 3 * W * (f.shared_ff or 0)
+        if L.latent is not None:
+            m = L.latent
+            linear += W * (m.heads * m.dim + m.kv_rank) + m.kv_rank * m.heads * (m.dim + m.vdim) + 2 * W * m.heads * m.vdim
+            total += sum(m.heads * 2 * (m.dim + m.vdim) * seen(t, m.window) for t in lens)
+        elif L.attention is not None:
+            a = L.attention
+            linear += W * ((a.heads + a.kv_heads) * 2 * a.dim + a.kv_heads * a.vdim + a.heads + a.heads * a.vdim)
+            total += sum(a.heads * 2 * 2 * (a.dim + a.vdim) * seen(t, None) for t in lens)
+        else:
+            r = L.retention
+            linear += W * r.heads * (2 * r.dim + 3 * r.vdim)
+            total += 6 * tokens * r.heads * r.dim * r.vdim
+        total += 2 * tokens * linear
+    return total + 2 * W * cfg.vocab * len(lens)
+
+
 def panodra_prefill_flops(cfg, lens) -> float:
     """The same count for a Panodra configuration, per layer run: the joint input projection, every head's keys and
     values from the latent, the output projection, causal attention per head over keys of dim + rot_dim and values of
@@ -378,6 +409,8 @@ def prefill_flops(cfg, lens) -> float:
         return pununex_prefill_flops(cfg, lens)
     if getattr(cfg, "architecture", "") == "Tosodra":
         return tosodra_prefill_flops(cfg, lens)
+    if getattr(cfg, "architecture", "") == "Zazulix":
+        return zazulix_prefill_flops(cfg, lens)
     if hasattr(cfg, "layers") and not hasattr(cfg, "hidden_size"):
         return lunulix_prefill_flops(cfg, lens)
     H, L, V = cfg.hidden_size, cfg.num_hidden_layers, cfg.vocab_size
@@ -547,7 +580,8 @@ def decode_kernel_times(lm, lens, seed: int):
              "ssd_scan", "ssd_group_norm", "token_gate", "gated_act", "attention_lse_gate", "add_dyt", "latent_kv_finish",
              "headwise", "latent_attention", "experts_few", "act_cast", "concat_cast", "logit_cap", "add_rmsnorm2", "head_finish",
              "attention_biased", "cols_cast", "delta_prep", "delta_scan", "delta_out", "gate_scale", "embed_bigram", "post_layernorm",
-             "add_layernorm", "route", "experts_identity", "sum_norm", "grouped_rmsnorm", "experts_dense", "experts_grouped_step", "conv_state_update"]
+             "add_layernorm", "route", "experts_identity", "sum_norm", "grouped_rmsnorm", "experts_dense", "experts_grouped_step", "conv_state_update",
+             "retention", "diff_combine"]
     names = [n for n in names if hasattr(K, n)]
     out, saved = {}, {n: getattr(K, n) for n in names}
     timing = [False]
@@ -582,14 +616,15 @@ def decode_kernel_times(lm, lens, seed: int):
     return {n: {"calls": c, "ms": round(ms, 4)} for n, (c, ms) in sorted(out.items(), key=lambda kv: -kv[1][1])}
 
 
-BESIDE = {"fuginex": "lunulix", "pununex": "fuginex", "tosodra": "pununex"}      # a design's closest other one (default: qwen3)
+BESIDE = {"fuginex": "lunulix", "pununex": "fuginex", "tosodra": "pununex", "zazulix": "pununex"}      # a design's closest other one (default: qwen3)
 
 
 def design_comparison(args) -> int:
-    """``--design lunulix`` / ``--design panodra`` / ``--design fuginex`` / ``--design pununex`` / ``--design tosodra``: decode and prefill
-    throughput of that design beside the closest other one (Qwen3; for Fuginex, Lunulix: an attention and a recurrence
+    """``--design lunulix`` / ``--design panodra`` / ``--design fuginex`` / ``--design pununex`` / ``--design tosodra`` /
+    ``--design zazulix``: decode and prefill throughput of that design beside the closest other one (Qwen3; for Fuginex, Lunulix: an attention and a recurrence
     side by side; for Pununex, Fuginex: a windowed attention beside a delta rule; for Tosodra, Pununex: norms behind the
-    sublayers, a bounded attention and routed experts) at equal width,
+    sublayers, a bounded attention and routed experts; for Zazulix, Pununex: recurrent layers, a windowed attention, dense
+    feed-forwards and routed experts by turns) at equal width,
     depth (layer runs), heads, feed-forward size and vocabulary (random weights), with where a step's time goes kernel by
     kernel."""
     import torch
@@ -650,7 +685,7 @@ def main() -> int:
     ap.add_argument("--repeats", type=int, default=5, help="timed regions of --steps steps; the median counts")
     ap.add_argument("--skip-points", action="store_true", help="leave out decode at batch 1 and 64 and the 32-bit check")
     ap.add_argument("--skip-sizes", action="store_true", help="leave out the points at 8B and 32B layer sizes")
-    ap.add_argument("--design", default="", choices=["", "lunulix", "panodra", "fuginex", "pununex", "tosodra"],
+    ap.add_argument("--design", default="", choices=["", "lunulix", "panodra", "fuginex", "pununex", "tosodra", "zazulix"],
                     help="instead of the default workload: this design beside its closest other one at equal layer sizes")
     ap.add_argument("--design-sizes", default="0.6b,8b", help="layer sizes of --design (presets <design>-<size>)")
     args = ap.parse_args()

@@ -20,6 +20,8 @@ def run(args) -> int:
         return latent_mixer(args, cfg)
     if args.kernel == "delta_mixer":
         return delta_mixer(args, cfg)
+    if args.kernel in ("retention_mixer", "differential_mixer"):
+        return mixer_alone(args, cfg, {"retention_mixer": "retention", "differential_mixer": "differential_attention"}[args.kernel])
     K = Kernels(torch.bfloat16, "cuda:0")
     # which kernel a product of many tokens takes (defaults: what the library chooses by itself)
     K.gemm_choices(pair=None if getattr(args, "pairs", None) is None else bool(args.pairs),
@@ -192,6 +194,43 @@ def delta_mixer(args, cfg) -> int:
             if i >= 3:
                 print(f"{name}, {B} x {T} tokens: {e0.elapsed_time(e1) * 1e3:.1f} us"
                       + (f" ({4 * B * T * H * dk * dv / 1e9:.2f} G multiply-adds)" if name != "delta mixer" else ""))
+    return 0
+
+
+def mixer_alone(args, cfg, kind: str) -> int:
+    """A preset's first mixer of a kind alone (``--size zazulix-0.6b``): ``--batch`` prompts of ``--context`` tokens, then single
+    tokens behind them; the whole mixer, with the L2 flushed between runs."""
+    from .cache import SequenceCache
+    from .engine.batch import context_from_packed, pack_step_host
+    from .kernels import Kernels
+    from .parts import MIXERS, Runtime
+    from .weights import random_weights
+    spec = next(L.mixer for L in cfg.to_model_spec().layers if L.mixer.kind == kind)
+    dev = torch.device("cuda:0")
+    rt = Runtime(device=dev, dtype=torch.bfloat16, kernels=Kernels(torch.bfloat16, dev))
+    cls = MIXERS.get(kind)
+    part = cls(spec, random_weights(cls.declare(spec, "m."), 1, 0.02, dtype=torch.bfloat16, device="cuda"), "m.", rt)
+    B, T = args.batch, args.context
+    cache = SequenceCache({0: cls.cache_need(spec)}, B * (T + 64), torch.bfloat16, "cuda:0", max_seqs=B, max_seq_len=T + 64)
+    slots = [cache.alloc_slot() for _ in range(B)]
+    cache.reserve([(s, T + 1) for s in slots]); cache.flush()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    for name, starts, lens in (("prompts", [0] * B, [T] * B), ("single tokens", [T] * B, [1] * B)):
+        x = torch.randn(sum(lens), spec.hidden, device="cuda").to(torch.bfloat16)
+        packed, n, q_lens = pack_step_host(slots, starts, [[0] * k for k in lens])
+        ctx = context_from_packed(packed.cuda(), n, slots, q_lens, starts)
+        ts = []
+        for i in range(args.reps + 3):
+            ctx.memo.clear()
+            flush.zero_()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            part.forward(x, ctx, cache.view(0), cache.state_of(0), True)
+            e1.record()
+            torch.cuda.synchronize()
+            if i >= 3:
+                ts.append(e0.elapsed_time(e1) * 1e3)
+        print(f"{kind}, {name}, {B} sequences of {T} tokens: {sorted(ts)[len(ts) // 2]:.1f} us")
     return 0
 
 
