@@ -632,3 +632,138 @@ def make_tosodra_dir(cfg: dict, out_dir: str, seed: int = 1, dtype=torch.bfloat1
         del f
         write_safetensors(path, tensors)
     return out_dir
+
+
+# ------------------------------------------------------------------------------------- Zazulix
+def zazulix_latent(heads=3, dim=16, vdim=24, kv_rank=40, scale=0.3, window=20, mlp="moe"):
+    """One ``latent_attention`` layer of a Zazulix config.json; ``mlp``: None, "moe", "dense", or a dict as config.json has it."""
+    m = dict(heads=heads, dim=dim, vdim=vdim, kv_rank=kv_rank, scale=scale)
+    if window:
+        m["mask"] = dict(size=window)
+    return dict(type="latent_attention", mixer=m, mlp=_zazulix_mlp(mlp))
+
+
+def zazulix_attention(heads=4, kv_heads=2, dim=12, vdim=20, scale=0.3, diff=0.4, conv=3, rot_dims=8, rot_base=5000.0, mlp="moe"):
+    m = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=scale, diff=diff)
+    if conv is not None:
+        m["conv"] = conv
+    if rot_dims:
+        m["rot"] = dict(base=rot_base, dims=rot_dims)
+    return dict(type="attention", mixer=m, mlp=_zazulix_mlp(mlp))
+
+
+def zazulix_retention(heads=3, dim=16, vdim=12, decay=(0.9, 0.995, 0.5), rot_dims=10, rot_base=7e3, mlp="dense"):
+    m = dict(heads=heads, dim=dim, vdim=vdim, decay=list(decay))
+    if rot_dims:
+        m["rot"] = dict(base=rot_base, dims=rot_dims)
+    return dict(type="retention", mixer=m, mlp=_zazulix_mlp(mlp))
+
+
+def zazulix_dense(ff=56, limit=0.8):
+    return dict(kind="dense", ff=ff, limit=limit)
+
+
+def zazulix_moe(experts=9, top=2, ff=24, groups=(3, 2), scale=1.4, shared=40):
+    r = dict(experts=experts, top=top, scale=scale)
+    if groups:
+        r["groups"] = dict(count=groups[0], keep=groups[1])
+    d = dict(kind="moe", expert=dict(ff=ff), router=r)
+    if shared:
+        d["shared"] = dict(ff=shared)
+    return d
+
+
+def _zazulix_mlp(mlp):
+    return zazulix_moe() if mlp == "moe" else zazulix_dense() if mlp == "dense" else mlp
+
+
+def zazulix_config(layers, vocab=91, width=32, eps=1e-5):
+    import copy
+    return dict(architecture="Zazulix", vocab=vocab, width=width, norm=dict(eps=eps), layers=[copy.deepcopy(L) for L in layers])
+
+
+# Small Zazulix models that differ from one another in every size and option.
+ZAZULIX = {
+    # every kind of layer and feed-forward, grouped heads, parts of a head turned, a layer without feed-forward
+    "A": lambda: zazulix_config([zazulix_attention(), zazulix_retention(), zazulix_latent(), zazulix_retention(
+        heads=2, dim=24, vdim=40, decay=(0.97, 1.0), rot_dims=24, mlp=None),
+        zazulix_attention(heads=6, kv_heads=1, dim=10, vdim=14, diff=0.1, conv=2, rot_dims=2,
+                          mlp=zazulix_moe(experts=8, top=4, ff=40, groups=(2, 1), shared=16)),
+        zazulix_latent(heads=5, window=70, vdim=16, mlp="dense")]),
+    # values of 1 and absent options: one head, one expert, one tap, a window of one key, nothing turned, no filter, no
+    # groups, no shared expert, a limit of 0, a head that does not fade
+    "B": lambda: zazulix_config([zazulix_latent(heads=1, dim=8, vdim=8, kv_rank=8, scale=1.0, window=1,
+                                                mlp=zazulix_moe(experts=1, top=1, ff=8, groups=None, scale=1.0, shared=8)),
+                                 zazulix_attention(heads=1, kv_heads=1, dim=4, vdim=8, scale=1.0, conv=1, rot_dims=0, diff=0.0,
+                                                   mlp=zazulix_moe(experts=4, top=1, ff=16, groups=(4, 1), shared=None)),
+                                 zazulix_retention(heads=1, dim=8, vdim=8, decay=(1.0,), rot_dims=0, mlp=zazulix_dense(8, 0.0)),
+                                 zazulix_attention(heads=2, kv_heads=2, dim=2, vdim=8, conv=None, rot_dims=2, mlp=None),
+                                 zazulix_latent(heads=1, dim=8, vdim=16, kv_rank=16, window=None, mlp=zazulix_dense(16, 5.0))],
+                                vocab=50, width=24),
+    # widths that are no multiple of 8 (bfloat16 rows off the 16-byte borders), odd head sizes, every expert chosen
+    "C": lambda: zazulix_config([zazulix_retention(heads=3, dim=10, vdim=7, decay=(0.8, 0.99, 0.999), rot_dims=6, mlp=zazulix_dense(30, 0.5)),
+                                 zazulix_attention(heads=3, kv_heads=3, dim=5, vdim=9, scale=0.4, conv=5, rot_dims=4, diff=0.7,
+                                                   mlp=zazulix_moe(experts=3, top=3, ff=12, groups=(1, 1), shared=20)),
+                                 zazulix_latent(heads=5, dim=6, vdim=10, kv_rank=22, window=65,
+                                                mlp=zazulix_moe(experts=6, top=2, ff=20, groups=(3, 3), shared=12))],
+                                vocab=33, width=20, eps=1e-6),
+    # head sizes the tensor-core attention has, windows of one page and of more than one, many experts, a retention wider
+    # than a tile
+    "T": lambda: zazulix_config([zazulix_attention(heads=4, kv_heads=1, dim=32, vdim=64, scale=0.2, conv=4, rot_dims=16,
+                                                   mlp=zazulix_moe(experts=12, top=3, ff=32, groups=(4, 2), shared=64)),
+                                 zazulix_retention(heads=2, dim=96, vdim=136, decay=(0.99, 0.9), rot_dims=96, mlp=zazulix_dense(96, 2.0)),
+                                 zazulix_latent(heads=4, dim=64, vdim=64, kv_rank=64, scale=0.2, window=64, mlp=None),
+                                 zazulix_attention(heads=2, kv_heads=2, dim=64, vdim=128, scale=0.15, conv=2, rot_dims=64, diff=0.8,
+                                                   mlp=zazulix_moe(experts=20, top=1, ff=64, groups=(2, 1), shared=32)),
+                                 zazulix_latent(heads=2, dim=48, vdim=80, kv_rank=96, scale=0.2, window=90)],
+                                vocab=211, width=96),
+}
+
+
+def zazulix_random_config(seed: int) -> dict:
+    """A Zazulix configuration drawn from sizes a model of the design may have: one to five layers of all kinds in any
+    order, grouped and ungrouped heads, windows below, at and above a page, part or all of a head turned, filters of
+    several lengths, experts in groups or not."""
+    import random
+    r = random.Random(seed)
+
+    def mlp():
+        kind = r.random()
+        if kind < 0.15:
+            return None
+        if kind < 0.4:
+            return zazulix_dense(ff=r.choice([48, 96, 200]), limit=r.choice([0.5, 1.0, 7.0]))
+        count = r.choice([1, 2, 4]); e = count * r.choice([1, 2, 3, 5]); keep = r.randint(1, count)
+        return zazulix_moe(experts=e, top=r.randint(1, min(4, keep * (e // count))), ff=r.choice([16, 40, 64]), groups=(count, keep),
+                           scale=r.choice([1.0, 2.5]), shared=r.choice([16, 32, 72]))
+
+    def layer():
+        kind = r.randrange(3)
+        if kind == 0:
+            return zazulix_latent(heads=r.choice([1, 2, 4, 6]), dim=r.choice([16, 32, 64, 128]), vdim=r.choice([16, 32, 64, 80]),
+                                  kv_rank=r.choice([32, 64, 96, 160]), scale=r.choice([0.1, 0.2, 0.15]),
+                                  window=r.choice([7, 48, 64, 70, 129, 200, 1000]), mlp=mlp())
+        if kind == 1:
+            h = r.choice([1, 2, 3, 5]); dim = r.choice([16, 32, 64, 100])
+            return zazulix_retention(heads=h, dim=dim, vdim=r.choice([16, 32, 64, 96]), decay=[1 - 2.0 ** -r.randint(1, 10) for _ in range(h)],
+                                     rot_dims=r.choice([2, 16, dim]), rot_base=r.choice([1e4, 1e6]), mlp=mlp())
+        kv = r.choice([1, 2, 4]); dim = r.choice([16, 32, 48, 64])
+        return zazulix_attention(heads=kv * r.choice([1, 2, 3]), kv_heads=kv, dim=dim, vdim=r.choice([2 * dim, 2 * dim, 16, 40]),
+                                 scale=r.choice([dim ** -0.5, 0.1, 0.2]), diff=r.choice([0.2, 0.5, 0.8]), conv=r.choice([2, 3, 4]),
+                                 rot_dims=r.choice([2, dim // 2, dim]), rot_base=r.choice([1e4, 4e5]), mlp=mlp())
+    return zazulix_config([layer() for _ in range(r.choice([1, 2, 3, 5]))], vocab=r.choice([128, 500, 1000]),
+                          width=r.choice([64, 96, 128, 240]), eps=r.choice([1e-5, 1e-6]))
+
+
+def make_zazulix_dir(cfg: dict, out_dir: str, seed: int = 1, dtype=torch.bfloat16, std: float = 0.15, edit=None) -> str:
+    """A Zazulix model folder with seeded random weights; ``edit(name, tensor) -> tensor`` may change them."""
+    from idempotent_llm_b200.config import ZazulixConfig
+    from idempotent_llm_b200.weights import write_random_model, write_safetensors, SafetensorsFile
+    write_random_model(ZazulixConfig.from_dict(cfg), out_dir, seed=seed, dtype=dtype, std=std)
+    if edit is not None:
+        path = os.path.join(out_dir, "model.safetensors")
+        f = SafetensorsFile(path)
+        tensors = [(n, edit(n, f.get(n).clone())) for n in f.names()]
+        del f
+        write_safetensors(path, tensors)
+    return out_dir
