@@ -138,83 +138,111 @@ __device__ __forceinline__ void rt_tile(float* dst, const float* __restrict__ sr
 }
 __device__ __forceinline__ void rt_wait() { asm volatile("cp.async.wait_all;\n" ::: "memory"); }
 
-// chunk_state[c, h, d, j] = sum_s g^(n-1-s) k_s[d] v_s[j]: a block per (chunk, head, 64 x 64 of the state), 4 x 4 of
-// them a thread
+// chunk_state[c, h, d, j] = sum_s g^(n-1-s) k_s[d] v_s[j]: a block per (chunk, head, 64 DT x 64 of the state), 4 DT x 4 of
+// them a thread (two tiles of dims share the values' reads)
+#define RT_STATE_SMEM(DT) (((DT) + 1) * RT_C * RT_LD * (int)sizeof(float))
+template <int DT>
 __global__ void __launch_bounds__(256) retention_chunk_state_kernel(RetentionArgs a) {
     pdl_launch_dependents();
     pdl_wait();
-    __shared__ __align__(16) float sk[RT_C * RT_LD];
-    __shared__ __align__(16) float sv[RT_C * RT_LD];
+    extern __shared__ __align__(16) float sm[];
+    float* sv = sm;
+    float* sk = sv + RT_C * RT_LD;                   // [DT] tiles
     __shared__ float pw[RT_C];
     const int c = blockIdx.x, h = blockIdx.y, tiles_j = (a.dv + 63) / 64;
-    const int d0 = blockIdx.z / tiles_j * 64, j0 = blockIdx.z % tiles_j * 64;
+    const int d0 = blockIdx.z / tiles_j * (64 * DT), j0 = blockIdx.z % tiles_j * 64;
     const int t0 = a.chunk_t0[c], n = a.chunk_t0[c + 1] - t0;
     const float* base = a.proj + (size_t)t0 * a.stride;
-    rt_tile(sk, base + a.col_k + h * a.dk + d0, a.stride, n, min(64, a.dk - d0), a.vec);
+#pragma unroll
+    for (int m = 0; m < DT; ++m)
+        rt_tile(sk + m * RT_C * RT_LD, base + a.col_k + h * a.dk + d0 + 64 * m, a.stride, n, min(64, a.dk - d0 - 64 * m), a.vec);
     rt_tile(sv, base + a.col_v + h * a.dv + j0, a.stride, n, min(64, a.dv - j0), a.vec);
     if (threadIdx.x < n) pw[threadIdx.x] = powf(a.decay[h], (float)(n - 1 - threadIdx.x));
     rt_wait();
     __syncthreads();
     const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
-    float acc[4][4];
+    float acc[DT][4][4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
-#pragma unroll
-        for (int k = 0; k < 4; ++k) acc[i][k] = 0.f;
-#pragma unroll 4
-    for (int t = 0; t < n; ++t) {
-        const float4 k4 = *reinterpret_cast<const float4*>(sk + t * RT_LD + ty * 4);
-        const float4 v4 = *reinterpret_cast<const float4*>(sv + t * RT_LD + tx * 4);
-        const float f = pw[t];
-        const float kx[4] = {k4.x * f, k4.y * f, k4.z * f, k4.w * f}, vx[4] = {v4.x, v4.y, v4.z, v4.w};
+    for (int m = 0; m < DT; ++m)
 #pragma unroll
         for (int i = 0; i < 4; ++i)
 #pragma unroll
-            for (int k = 0; k < 4; ++k) acc[i][k] = fmaf(kx[i], vx[k], acc[i][k]);
+            for (int k = 0; k < 4; ++k) acc[m][i][k] = 0.f;
+#pragma unroll 4
+    for (int t = 0; t < n; ++t) {
+        float4 v4 = *reinterpret_cast<const float4*>(sv + t * RT_LD + tx * 4);
+        const float f = pw[t];
+        const float vx[4] = {v4.x * f, v4.y * f, v4.z * f, v4.w * f};
+#pragma unroll
+        for (int m = 0; m < DT; ++m) {
+            const float4 k4 = *reinterpret_cast<const float4*>(sk + (m * RT_C + t) * RT_LD + ty * 4);
+            const float kx[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int k = 0; k < 4; ++k) acc[m][i][k] = fmaf(kx[i], vx[k], acc[m][i][k]);
+        }
     }
     float* dst = a.chunk_state + ((size_t)c * a.H + h) * a.dk * a.dv;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-        const int d = d0 + ty * 4 + i, j = j0 + tx * 4;
-        if (d >= a.dk) break;
-        float* p = dst + (size_t)d * a.dv + j;
-        if (a.vec && j + 4 <= a.dv) {
-            *reinterpret_cast<float4*>(p) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
-        } else {
+    for (int m = 0; m < DT; ++m)
 #pragma unroll
-            for (int k = 0; k < 4; ++k)
-                if (j + k < a.dv) p[k] = acc[i][k];
+        for (int i = 0; i < 4; ++i) {
+            const int d = d0 + 64 * m + ty * 4 + i, j = j0 + tx * 4;
+            if (d >= a.dk) break;
+            float* p = dst + (size_t)d * a.dv + j;
+            if (a.vec && j + 4 <= a.dv) {
+                *reinterpret_cast<float4*>(p) = make_float4(acc[m][i][0], acc[m][i][1], acc[m][i][2], acc[m][i][3]);
+            } else {
+#pragma unroll
+                for (int k = 0; k < 4; ++k)
+                    if (j + k < a.dv) p[k] = acc[m][i][k];
+            }
         }
-    }
 }
 
-// chunk after chunk: what a chunk starts from takes the place of what it adds, and the state moves on
+// chunk after chunk: what a chunk starts from takes the place of what it adds, and the state moves on.  A thread has V
+// elements side by side; the chunks of a batch are on their way together, only the sums are a chain.
 #define RT_BATCH 8
-__global__ void __launch_bounds__(256) retention_carry_kernel(RetentionArgs a) {
+template <int V>
+__global__ void __launch_bounds__(128) retention_carry_kernel(RetentionArgs a) {
     pdl_launch_dependents();
     pdl_wait();
     const int s = blockIdx.z, h = blockIdx.y;
-    const size_t per = (size_t)a.dk * a.dv, e = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (e >= per) return;
+    const size_t per = (size_t)a.dk * a.dv, e = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
+    if (e >= per) return;                                       // (V == 4: dv is a multiple of 4)
     const int c0 = a.seq_chunk0[s], c1 = a.seq_chunk0[s + 1];
     float* st = a.state + (size_t)a.slots[s] * a.state_stride + (size_t)h * per + e;
     float* cs = a.chunk_state + ((size_t)c0 * a.H + h) * per + e;
     const size_t step = (size_t)a.H * per;
     const float g = a.decay[h], whole = powf(g, (float)RT_C);
-    float S = *st;
-    for (int b = c0; b < c1; b += RT_BATCH, cs += RT_BATCH * step) {
-        float add[RT_BATCH];
+    // every chunk of a portion but its last is whole
+    const float last = c1 > c0 ? powf(g, (float)(a.chunk_t0[c1] - a.chunk_t0[c1 - 1])) : 1.f;
+    float S[V];
 #pragma unroll
-        for (int u = 0; u < RT_BATCH; ++u) add[u] = b + u < c1 ? cs[u * step] : 0.f;
+    for (int i = 0; i < V; ++i) S[i] = st[i];
+    for (int b = c0; b < c1; b += RT_BATCH, cs += RT_BATCH * step) {
+        float add[RT_BATCH][V];
 #pragma unroll
         for (int u = 0; u < RT_BATCH; ++u)
             if (b + u < c1) {
-                cs[u * step] = S;
-                const int n = a.chunk_t0[b + u + 1] - a.chunk_t0[b + u];
-                S = fmaf(n == RT_C ? whole : powf(g, (float)n), S, add[u]);
+                if constexpr (V == 4) {
+                    const float4 x = *reinterpret_cast<const float4*>(cs + u * step);
+                    add[u][0] = x.x; add[u][1] = x.y; add[u][2] = x.z; add[u][3] = x.w;
+                } else add[u][0] = cs[u * step];
+            }
+#pragma unroll
+        for (int u = 0; u < RT_BATCH; ++u)
+            if (b + u < c1) {
+                if constexpr (V == 4) *reinterpret_cast<float4*>(cs + u * step) = make_float4(S[0], S[1], S[2], S[3]);
+                else cs[u * step] = S[0];
+                const float f = b + u + 1 < c1 ? whole : last;
+#pragma unroll
+                for (int i = 0; i < V; ++i) S[i] = fmaf(f, S[i], add[u][i]);
             }
     }
-    *st = S;
+#pragma unroll
+    for (int i = 0; i < V; ++i) st[i] = S[i];
 }
 
 // read-outs: a block per (chunk, head, 64 columns); per 64 dims of the keys it adds q k^T to the chunk's pair scores and
@@ -236,6 +264,7 @@ __global__ void __launch_bounds__(256) retention_chunk_out_kernel(RetentionArgs 
     if (threadIdx.x <= RT_C) pw[threadIdx.x] = powf(a.decay[h], (float)threadIdx.x);
     rt_tile(sv, base + a.col_v + h * a.dv + j0, a.stride, n, nj, a.vec);
     const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+    const int nk = (4 * (ty | 1) + 3) / 16 + 1;      // groups of 16 tokens that a warp's rows (two ty) may see
     float pair[4][4], out[4][4];                     // pair[i][k]: tokens t = 4 ty + i, s = tx + 16 k;  out[i][k]: column 4 tx + k
 #pragma unroll
     for (int i = 0; i < 4; ++i)
@@ -256,6 +285,7 @@ __global__ void __launch_bounds__(256) retention_chunk_out_kernel(RetentionArgs 
             for (int i = 0; i < 4; ++i) q4[i] = *reinterpret_cast<const float4*>(sq + (4 * ty + i) * RT_LD + d);
 #pragma unroll
             for (int k = 0; k < 4; ++k) {
+                if (k >= nk) break;                  // (a warp's rows all lie before these tokens)
                 const float4 k4 = *reinterpret_cast<const float4*>(sk + (tx + 16 * k) * RT_LD + d);
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
@@ -323,7 +353,7 @@ extern "C" int idm_retention_chunk_tokens() { return RT_C; }
 extern "C" long long idm_retention_scratch_floats(int n_chunks, int H, int dk, int dv) { return (long long)n_chunks * H * dk * dv; }
 
 // chunk_t0 [n_chunks + 1], seq_chunk0 [n_seqs + 1] as for the other chunked recurrence (a chunk ends where the next
-// begins, chunks hold at most RT_C tokens and never cross a sequence's border); n_chunks == 0: every sequence token by
+// begins, chunks hold RT_C tokens, a sequence's last one up to so many, and never cross a sequence's border); n_chunks == 0: every sequence token by
 // token.  In chunks, the step's q and k columns of `proj` are turned in place.
 extern "C" int idm_retention(float* proj, int stride, int col_q, int col_k, int col_v, const float* cs, int half, float k_scale,
                              const float* decay, float* state, long long state_stride, float* o, int o_stride, const int* cu_q,
@@ -356,16 +386,25 @@ extern "C" int idm_retention(float* proj, int stride, int col_q, int col_k, int 
     const int items = 2 * H * (dk - half), tiles_d = (dk + 63) / 64, tiles_j = (dv + 63) / 64;
     idm_launch(retention_turn_kernel, dim3(n_tokens, min(8, (items + 255) / 256)), dim3(256), 0, stream, a);
     IDM_LAUNCH_CHECK("retention_turn");
-    idm_launch(retention_chunk_state_kernel, dim3(n_chunks, H, tiles_d * tiles_j), dim3(256), 0, stream, a);
-    IDM_LAUNCH_CHECK("retention_chunk_state");
-    idm_launch(retention_carry_kernel, dim3((unsigned)(((size_t)dk * dv + 255) / 256), H, n_seqs), dim3(256), 0, stream, a);
-    IDM_LAUNCH_CHECK("retention_carry");
     static bool set = false;
     if (!set) {
         cudaError_t e = cudaFuncSetAttribute(retention_chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, RT_OUT_SMEM);
+        if (e == cudaSuccess)
+            e = cudaFuncSetAttribute(retention_chunk_state_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, RT_STATE_SMEM(2));
         IDM_REQUIRE(e == cudaSuccess, "retention: %d bytes of shared memory were refused (%s)", RT_OUT_SMEM, cudaGetErrorString(e));
         set = true;
     }
+    if (tiles_d > 1)
+        idm_launch(retention_chunk_state_kernel<2>, dim3(n_chunks, H, (tiles_d + 1) / 2 * tiles_j), dim3(256), RT_STATE_SMEM(2), stream, a);
+    else
+        idm_launch(retention_chunk_state_kernel<1>, dim3(n_chunks, H, tiles_j), dim3(256), RT_STATE_SMEM(1), stream, a);
+    IDM_LAUNCH_CHECK("retention_chunk_state");
+    const size_t per = (size_t)dk * dv;
+    if (a.vec)
+        idm_launch(retention_carry_kernel<4>, dim3((unsigned)((per / 4 + 127) / 128), H, n_seqs), dim3(128), 0, stream, a);
+    else
+        idm_launch(retention_carry_kernel<1>, dim3((unsigned)((per + 127) / 128), H, n_seqs), dim3(128), 0, stream, a);
+    IDM_LAUNCH_CHECK("retention_carry");
     idm_launch(retention_chunk_out_kernel, dim3(n_chunks, H, tiles_j), dim3(256), RT_OUT_SMEM, stream, a);
     IDM_LAUNCH_CHECK("retention_chunk_out");
     return 0;
