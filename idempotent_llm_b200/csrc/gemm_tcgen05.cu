@@ -93,22 +93,29 @@ __device__ __forceinline__ void trace_stamp(int) {}
 __device__ __forceinline__ void block_stamp(int, int) {}
 #endif
 
-enum { EPI_STORE = 1, EPI_RESIDUAL = 2, EPI_SWIGLU = 3, EPI_QKV = 4 };
+// SWIGLU is silu alone; GATED has every activation, their constants and the factors per row (an epilogue of its own: what a
+// few-token product spends on fetching instructions it does not need shows in a step)
+enum { EPI_STORE = 1, EPI_RESIDUAL = 2, EPI_SWIGLU = 3, EPI_QKV = 4, EPI_GATED = 5 };
 
 struct GemmEpi {
     float* out;          // STORE: [M, N]; RESIDUAL: the residual stream [M, N]
-    T* y; int inter;     // SWIGLU: y [M, inter]
-    int act;             // SWIGLU: which gated activation (gated_act in common.cuh; 0 = silu)
-    float limit, slope;  // SWIGLU: the constants of the clamped activation
-    const float* row_w;  // SWIGLU, or null: row_w[t] multiplies gate and up of token t before the activation
-    const float* row_out;    // SWIGLU, or null: row_out[t] multiplies what the activation gives
+    T* y; int inter;     // SWIGLU, GATED: y [M, inter]
+    int act;             // GATED: which gated activation (gated_act in common.cuh)
+    float limit, slope;  // GATED: the constants of the clamped activation
+    const float* row_w;  // GATED, or null: row_w[t] multiplies gate and up of token t before the activation
+    const float* row_out;    // GATED, or null: row_out[t] multiplies what the activation gives
     QkvArgs q;           // QKV
 };
 
 // four features of the gated activation from (gate, up) pairs side by side
-__device__ __forceinline__ void gated_act4(float* y, float4 a, float4 b, const GemmEpi& e) {
-    y[0] = gated_act(a.x, a.y, e.act, e.limit, e.slope); y[1] = gated_act(a.z, a.w, e.act, e.limit, e.slope);
-    y[2] = gated_act(b.x, b.y, e.act, e.limit, e.slope); y[3] = gated_act(b.z, b.w, e.act, e.limit, e.slope);
+template <int EPI>
+__device__ __forceinline__ float epi_act(float g, float u, const GemmEpi& e) {
+    return EPI == EPI_SWIGLU ? silu_mul(g, u) : gated_act(g, u, e.act, e.limit, e.slope);
+}
+template <int EPI>
+__device__ __forceinline__ void epi_act4(float* y, float4 a, float4 b, const GemmEpi& e) {
+    y[0] = epi_act<EPI>(a.x, a.y, e); y[1] = epi_act<EPI>(a.z, a.w, e);
+    y[2] = epi_act<EPI>(b.x, b.y, e); y[3] = epi_act<EPI>(b.z, b.w, e);
 }
 
 // ------------------------------------------------------------------- persistent kernel (many tokens)
@@ -195,22 +202,22 @@ __device__ __forceinline__ void persistent_tile_epilogue(const GemmEpi& e, uint3
 #pragma unroll
             for (int j = 0; j < GP_CHUNK; ++j) xs[j * GT_BM + fl] = v[j];
             group_sync(grp);
-            if (EPI == EPI_SWIGLU) {
+            if (EPI == EPI_SWIGLU || EPI == EPI_GATED) {
                 // 8 consecutive features of y (16 tile rows: gate, up, gate, up, ...) per thread, one
                 // 16-byte store; the group's 128 threads cover the chunk's 16 token rows
                 const int j = fl >> 3, sub = fl & 7;
                 if (j < cols) {
                     const float4* src = reinterpret_cast<const float4*>(xs + j * GT_BM + sub * 16);
                     float4 p0 = src[0], p1 = src[1], p2 = src[2], p3 = src[3];
-                    if (e.row_w) {
+                    if (EPI == EPI_GATED && e.row_w) {
                         const float rw = e.row_w[t0 + c0 + j];
                         p0.x *= rw; p0.y *= rw; p0.z *= rw; p0.w *= rw; p1.x *= rw; p1.y *= rw; p1.z *= rw; p1.w *= rw;
                         p2.x *= rw; p2.y *= rw; p2.z *= rw; p2.w *= rw; p3.x *= rw; p3.y *= rw; p3.z *= rw; p3.w *= rw;
                     }
                     float y8[8];
-                    gated_act4(y8, p0, p1, e);
-                    gated_act4(y8 + 4, p2, p3, e);
-                    if (e.row_out) {
+                    epi_act4<EPI>(y8, p0, p1, e);
+                    epi_act4<EPI>(y8 + 4, p2, p3, e);
+                    if (EPI == EPI_GATED && e.row_out) {
                         const float ro = e.row_out[t0 + c0 + j];
 #pragma unroll
                         for (int i = 0; i < 8; ++i) y8[i] = __fmul_rn(y8[i], ro);
@@ -885,7 +892,7 @@ __global__ void __launch_bounds__(GS_THREADS) gemm_small_kernel(const __grid_con
     const int f0 = blockIdx.x * bf;
     const int t0 = blockIdx.y * 128;                             // more than 128 tokens: a block per 128 of them (and slice)
     const int n_groups = (kb_total + gk - 1) / gk;
-    if (threadIdx.x == 0) block_stamp(EPI == EPI_RESIDUAL ? (kb_total > 32 ? 1 : 0) : EPI == EPI_SWIGLU ? 2 : EPI == EPI_QKV ? 3 : 4, 4);   // the block is there
+    if (threadIdx.x == 0) block_stamp(EPI == EPI_RESIDUAL ? (kb_total > 32 ? 1 : 0) : EPI == EPI_SWIGLU || EPI == EPI_GATED ? 2 : EPI == EPI_QKV ? 3 : 4, 4);   // the block is there
 
     if (threadIdx.x == 0) {
         for (int s = 0; s < stages; ++s) { mbar_init(full_bar(s), 1); mbar_init(empty_bar(s), 1); }
@@ -900,11 +907,11 @@ __global__ void __launch_bounds__(GS_THREADS) gemm_small_kernel(const __grid_con
     const uint32_t tmem_d = *tmem_slot;
 #if defined(IDM_TRACE)
     // (stamps of the four fused products of a layer side by side: residual with a short / long inner axis, SwiGLU, q/k/v)
-    if (blockIdx.x == 0 && threadIdx.x == 0) g_gemm_trace_base = EPI == EPI_RESIDUAL ? (kb_total > 32 ? 10 : 0) : EPI == EPI_SWIGLU ? 20 : EPI == EPI_QKV ? 30 : 40;
+    if (blockIdx.x == 0 && threadIdx.x == 0) g_gemm_trace_base = EPI == EPI_RESIDUAL ? (kb_total > 32 ? 10 : 0) : EPI == EPI_SWIGLU || EPI == EPI_GATED ? 20 : EPI == EPI_QKV ? 30 : 40;
     __syncthreads();
 #endif
     if (threadIdx.x == 0) trace_stamp(0);                        // set-up done
-    const int trace_kind = EPI == EPI_RESIDUAL ? (kb_total > 32 ? 1 : 0) : EPI == EPI_SWIGLU ? 2 : EPI == EPI_QKV ? 3 : 4;
+    const int trace_kind = EPI == EPI_RESIDUAL ? (kb_total > 32 ? 1 : 0) : EPI == EPI_SWIGLU || EPI == EPI_GATED ? 2 : EPI == EPI_QKV ? 3 : 4;
 
     if (warp == 4) {
         // ------------------------------------------------------------ TMA producer
@@ -1055,11 +1062,11 @@ __global__ void __launch_bounds__(GS_THREADS) gemm_small_kernel(const __grid_con
                                 if (f0 + c0 + j < n_features) p[j] = EPI == EPI_RESIDUAL ? p[j] + v[j] : v[j];
                         }
                     }
-                } else if (EPI == EPI_SWIGLU) {
+                } else if (EPI == EPI_SWIGLU || EPI == EPI_GATED) {
                     // the tile's columns are gate, up, gate, up, ... of the features f0 / 2 ..; 32 columns are asked
                     // for before the first is waited for
-                    const float rw = e.row_w && live ? e.row_w[t] : 1.0f;      // (a factor of 1 changes no bit)
-                    const float ro = e.row_out && live ? e.row_out[t] : 1.0f;
+                    const float rw = EPI == EPI_GATED && e.row_w && live ? e.row_w[t] : 1.0f;      // (a factor of 1 changes no bit)
+                    const float ro = EPI == EPI_GATED && e.row_out && live ? e.row_out[t] : 1.0f;
 #pragma unroll 1
                     for (int c0 = 0; c0 < bf; c0 += 32) {
                         if (((f0 + c0) >> 1) >= e.inter) break;
@@ -1075,8 +1082,9 @@ __global__ void __launch_bounds__(GS_THREADS) gemm_small_kernel(const __grid_con
                             float y8[8];
 #pragma unroll
                             for (int i = 0; i < 8; ++i)
-                                y8[i] = __fmul_rn(gated_act(__fmul_rn(__uint_as_float(raw[16 * h + 2 * i]), rw), __fmul_rn(__uint_as_float(raw[16 * h + 2 * i + 1]), rw), e.act,
-                                                            e.limit, e.slope), ro);
+                                y8[i] = EPI == EPI_SWIGLU ? silu_mul(__uint_as_float(raw[16 * h + 2 * i]), __uint_as_float(raw[16 * h + 2 * i + 1]))
+                                                          : __fmul_rn(epi_act<EPI>(__fmul_rn(__uint_as_float(raw[16 * h + 2 * i]), rw),
+                                                                                   __fmul_rn(__uint_as_float(raw[16 * h + 2 * i + 1]), rw), e), ro);
                             T* dst = e.y + (size_t)t * e.inter + fg;
                             if ((e.inter & 7) == 0 && fg + 8 <= e.inter) {
                                 store8(dst, y8);
@@ -1472,10 +1480,11 @@ extern "C" int idm_gemm_bf16_swiglu(const void* x, const void* w_tiled, void* y,
 extern "C" int idm_gemm_bf16_gated_all(const void* x, const void* w_tiled, void* y, int M, int inter, int K, int act,
                                        float limit, float slope, const float* row_w, const float* row_out, cudaStream_t stream) {
     IDM_REQUIRE(act >= 0 && act <= IDM_ACT_CLAMPED, "gemm_gated: activation %d is not built", act);
+    if (act == 0 && row_w == nullptr && row_out == nullptr) return idm_gemm_bf16_swiglu(x, w_tiled, y, M, inter, K, stream);
     GemmEpi e = {};
     e.y = (T*)y; e.inter = inter; e.act = act; e.row_w = row_w; e.row_out = row_out; e.limit = limit; e.slope = slope;
     const int tiles = (inter + 63) / 64;
-    return gemm_any<EPI_SWIGLU>(x, w_tiled, e, M, tiles * GT_BM, K, stream);
+    return gemm_any<EPI_GATED>(x, w_tiled, e, M, tiles * GT_BM, K, stream);
 }
 
 extern "C" int idm_gemm_bf16_gated_rows(const void* x, const void* w_tiled, void* y, int M, int inter, int K, int act,
